@@ -30,16 +30,18 @@ RELEASED = 0   # block-table entry of a page the window has passed: the scratch 
 @dataclass(frozen=True)
 class GroupSpec:
     """A group of layers with the same need: ``window`` and ``chunk`` None keeps all positions, ``window`` the last
-    that many, ``chunk`` those of the newest token's own block of that many positions (counted from position 0)."""
+    that many, ``chunk`` those of the newest token's own block of that many positions (counted from position 0); the pages
+    that hold the first ``keep`` positions are never given back while the request lives."""
     name: str
     window: int | None = None
     chunk: int | None = None
+    keep: int = 0
 
 
 @dataclass
 class RequestCache:
     """What one request holds.  ``tables[g][i]`` is the physical page of logical page i in
-    group g; ``first_live[g]`` is the first logical page not yet released."""
+    group g; ``first_live[g]`` is the first logical page not yet released (kept first pages aside)."""
     tables: list = field(default_factory=list)
     first_live: list = field(default_factory=list)
     state_slot: int = 0
@@ -137,7 +139,8 @@ class CacheManager:
             return released
         for g in range(len(self.groups)):
             first = min(self._first_needed_page(g, rc.num_computed), len(rc.tables[g]))
-            for i in range(rc.first_live[g], first):
+            kept = -(-self.groups[g].keep // self.block_size)          # pages with kept first positions stay
+            for i in range(max(rc.first_live[g], kept), first):
                 p = rc.tables[g][i]
                 if p != RELEASED:
                     released[g].append(p)

@@ -46,17 +46,20 @@ class CacheLayout:
 
         for layer, n in needs.items():
             add(layer, n)
-        kinds = sorted({(n.window, n.chunk) for n in flat.values() if isinstance(n, KVNeed)},
-                       key=lambda wc: (wc[0] is not None, wc[0] or 0, wc[1] is not None, wc[1] or 0))
+        # (a layer that keeps every position keeps the first ones too: ``keep`` tells groups apart only beside a window or block)
+        kind_of = lambda n: (n.window, n.chunk, n.keep if n.window is not None or n.chunk is not None else 0)
+        kinds = sorted({kind_of(n) for n in flat.values() if isinstance(n, KVNeed)},
+                       key=lambda wck: (wck[0] is not None, wck[0] or 0, wck[1] is not None, wck[1] or 0, wck[2]))
         index = {}
-        for w, c in kinds:
+        for w, c, keep in kinds:
             if w is not None and c is not None:
                 raise ValueError("a layer keeps a window or a block of positions, not both")
-            index[(w, c)] = len(lay.groups)
-            lay.groups.append(GroupSpec("full" if w is None and c is None else (f"window{w}" if c is None else f"chunk{c}"), w, c))
+            index[(w, c, keep)] = len(lay.groups)
+            name = "full" if w is None and c is None else (f"window{w}" if c is None else f"chunk{c}")
+            lay.groups.append(GroupSpec(name + (f"+first{keep}" if keep else ""), w, c, keep))
         for layer, n in flat.items():
             if isinstance(n, KVNeed):
-                lay.kv[layer] = (index[(n.window, n.chunk)], n)
+                lay.kv[layer] = (index[kind_of(n)], n)
             elif isinstance(n, StateNeed):
                 lay.state[layer] = n
             elif n is not None:

@@ -7,6 +7,7 @@ from __future__ import annotations
 from .getizen_config import GetizenConfig
 from .kebudra_config import KebudraConfig
 from .luluzen_config import LuluzenConfig
+from .radenex_config import RadenexConfig
 from .serotar_config import SerotarConfig
 from .model_config import ConfigError, LlamaConfig, read_config_json
 
@@ -46,6 +47,7 @@ register_architecture("Getizen", GetizenConfig)
 register_architecture("Kebudra", KebudraConfig)
 register_architecture("Serotar", SerotarConfig)
 register_architecture("Luluzen", LuluzenConfig)
+register_architecture("Radenex", RadenexConfig)
 
 
 def preset_names() -> list[str]:

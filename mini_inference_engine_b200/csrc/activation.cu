@@ -167,10 +167,10 @@ extern "C" int mie_glu_clamped(const void* gu, void* out, int act_tag, int num_t
 
 // An output gate on attention heads: out[t, h * Dv + c] = attn[t, h, c] * sigmoid(g[t, h * Dv + c]) for c < Dv, where
 // attn rows hold H heads of DP >= Dv entries (the padded tail is dropped) and g is a part of a fused projection
-// with row stride `g_stride`.
+// with row stride `g_stride`.  `per_head`: one gate logit a head, g[t, h].
 template <typename T>
 __global__ void sigmoid_gate_kernel(const T* __restrict__ attn, const T* __restrict__ g, int64_t g_stride, T* __restrict__ out,
-                                    int64_t total, int H, int Dv, int DP) {
+                                    int64_t total, int H, int Dv, int DP, int per_head) {
     pdl_enter();
     const int n = H * Dv;
     for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
@@ -178,13 +178,13 @@ __global__ void sigmoid_gate_kernel(const T* __restrict__ attn, const T* __restr
         const int64_t t = idx / n;
         const int i = (int)(idx - t * n);
         const int h = i / Dv, c = i - h * Dv;
-        const float z = to_f32<T>(g[t * g_stride + i]);
+        const float z = to_f32<T>(g[t * g_stride + (per_head ? h : i)]);
         out[idx] = from_f32<T>(to_f32<T>(attn[(t * H + h) * DP + c]) / (1.0f + expf(-z)));
     }
 }
 
 __global__ void sigmoid_gate_bf16x8_kernel(const bf16* __restrict__ attn, const bf16* __restrict__ g, int64_t g_stride,
-                                           bf16* __restrict__ out, int64_t total8, int H, int Dv8, int DP) {
+                                           bf16* __restrict__ out, int64_t total8, int H, int Dv8, int DP, int per_head) {
     pdl_enter();
     const int n8 = H * Dv8;
     for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total8; idx += (int64_t)gridDim.x * blockDim.x) {
@@ -192,11 +192,18 @@ __global__ void sigmoid_gate_bf16x8_kernel(const bf16* __restrict__ attn, const 
         const int i8 = (int)(idx - t * n8);
         const int h = i8 / Dv8, c8 = i8 - h * Dv8;
         const uint4 a = *reinterpret_cast<const uint4*>(attn + (t * H + h) * DP + 8 * c8);
-        const uint4 z = *reinterpret_cast<const uint4*>(g + t * g_stride + 8 * i8);
         const __nv_bfloat162* ha = reinterpret_cast<const __nv_bfloat162*>(&a);
-        const __nv_bfloat162* hz = reinterpret_cast<const __nv_bfloat162*>(&z);
         uint4 o;
         __nv_bfloat162* ho = reinterpret_cast<__nv_bfloat162*>(&o);
+        if (per_head) {
+            const float s = __fdividef(1.0f, 1.0f + __expf(-__bfloat162float(g[t * g_stride + h])));
+#pragma unroll
+            for (int j = 0; j < 4; ++j) { const float2 x = __bfloat1622float2(ha[j]); ho[j] = __floats2bfloat162_rn(x.x * s, x.y * s); }
+            *reinterpret_cast<uint4*>(out + idx * 8) = o;
+            continue;
+        }
+        const uint4 z = *reinterpret_cast<const uint4*>(g + t * g_stride + 8 * i8);
+        const __nv_bfloat162* hz = reinterpret_cast<const __nv_bfloat162*>(&z);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const float2 x = __bfloat1622float2(ha[j]), y = __bfloat1622float2(hz[j]);
@@ -207,24 +214,24 @@ __global__ void sigmoid_gate_bf16x8_kernel(const bf16* __restrict__ attn, const 
 }
 
 extern "C" int mie_sigmoid_gate(const void* attn, const void* g, long long g_stride, void* out, int act_tag, int num_tokens,
-                                int H, int Dv, int DP, cudaStream_t stream) {
+                                int H, int Dv, int DP, int per_head, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (H <= 0 || Dv <= 0 || DP < Dv) return MIE_ERR_BAD_ARG;
     const int64_t total = (int64_t)num_tokens * H * Dv;
     const int threads = 256;
-    if (act_tag == MIE_BF16 && Dv % 8 == 0 && DP % 8 == 0 && g_stride % 8 == 0 &&
-        (reinterpret_cast<uintptr_t>(attn) | reinterpret_cast<uintptr_t>(g) | reinterpret_cast<uintptr_t>(out)) % 16 == 0) {
+    if (act_tag == MIE_BF16 && Dv % 8 == 0 && DP % 8 == 0 && (per_head || g_stride % 8 == 0) &&
+        (reinterpret_cast<uintptr_t>(attn) | (per_head ? 0 : reinterpret_cast<uintptr_t>(g)) | reinterpret_cast<uintptr_t>(out)) % 16 == 0) {
         int64_t blocks8 = (total / 8 + threads - 1) / threads;
         if (blocks8 > device_sm_count() * 16) blocks8 = device_sm_count() * 16;
         return launch_kernel(sigmoid_gate_bf16x8_kernel, dim3((int)blocks8), dim3(threads), 0, stream, (const bf16*)attn, (const bf16*)g,
-                             (int64_t)g_stride, (bf16*)out, total / 8, H, Dv / 8, DP);
+                             (int64_t)g_stride, (bf16*)out, total / 8, H, Dv / 8, DP, per_head);
     }
     int64_t blocks = (total + threads - 1) / threads;
     if (blocks > device_sm_count() * 16) blocks = device_sm_count() * 16;
     if (act_tag == MIE_F32)
-        return launch_kernel(sigmoid_gate_kernel<float>, dim3((int)blocks), dim3(threads), 0, stream, (const float*)attn, (const float*)g, (int64_t)g_stride, (float*)out, total, H, Dv, DP);
+        return launch_kernel(sigmoid_gate_kernel<float>, dim3((int)blocks), dim3(threads), 0, stream, (const float*)attn, (const float*)g, (int64_t)g_stride, (float*)out, total, H, Dv, DP, per_head);
     else if (act_tag == MIE_BF16)
-        return launch_kernel(sigmoid_gate_kernel<bf16>, dim3((int)blocks), dim3(threads), 0, stream, (const bf16*)attn, (const bf16*)g, (int64_t)g_stride, (bf16*)out, total, H, Dv, DP);
+        return launch_kernel(sigmoid_gate_kernel<bf16>, dim3((int)blocks), dim3(threads), 0, stream, (const bf16*)attn, (const bf16*)g, (int64_t)g_stride, (bf16*)out, total, H, Dv, DP, per_head);
     return MIE_ERR_BAD_ARG;
 }
 
@@ -268,6 +275,44 @@ extern "C" int mie_xielu(const void* x, void* out, int act_tag, long long total,
         return launch_kernel(xielu_kernel<float>, dim3((int)blocks), dim3(threads), 0, stream, (const float*)x, (float*)out, (int64_t)total, ap, an);
     else if (act_tag == MIE_BF16)
         return launch_kernel(xielu_kernel<bf16>, dim3((int)blocks), dim3(threads), 0, stream, (const bf16*)x, (bf16*)out, (int64_t)total, ap, an);
+    return MIE_ERR_BAD_ARG;
+}
+
+// The square of relu, max(z, 0)^2, elementwise.
+template <typename T>
+__global__ void relu2_kernel(const T* __restrict__ x, T* __restrict__ out, int64_t total) {
+    pdl_enter();
+    for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (int64_t)gridDim.x * blockDim.x) {
+        const float z = fmaxf(to_f32<T>(x[idx]), 0.f);
+        out[idx] = from_f32<T>(z * z);
+    }
+}
+__global__ void relu2_bf16x8_kernel(const bf16* __restrict__ x, bf16* __restrict__ out, int64_t total8) {
+    pdl_enter();
+    for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total8; idx += (int64_t)gridDim.x * blockDim.x) {
+        uint4 u = *reinterpret_cast<const uint4*>(x + idx * 8);
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            float2 f = __bfloat1622float2(h[j]);
+            f.x = fmaxf(f.x, 0.f); f.y = fmaxf(f.y, 0.f);
+            h[j] = __floats2bfloat162_rn(f.x * f.x, f.y * f.y);
+        }
+        *reinterpret_cast<uint4*>(out + idx * 8) = u;
+    }
+}
+
+extern "C" int mie_relu2(const void* x, void* out, int act_tag, long long total, cudaStream_t stream) {
+    if (total <= 0) return 0;
+    const int threads = 256;
+    const bool vec = act_tag == MIE_BF16 && total % 8 == 0 && (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+    int64_t blocks = ((vec ? total / 8 : total) + threads - 1) / threads;
+    if (blocks > device_sm_count() * 16) blocks = device_sm_count() * 16;
+    if (vec) return launch_kernel(relu2_bf16x8_kernel, dim3((int)blocks), dim3(threads), 0, stream, (const bf16*)x, (bf16*)out, (int64_t)(total / 8));
+    if (act_tag == MIE_F32)
+        return launch_kernel(relu2_kernel<float>, dim3((int)blocks), dim3(threads), 0, stream, (const float*)x, (float*)out, (int64_t)total);
+    else if (act_tag == MIE_BF16)
+        return launch_kernel(relu2_kernel<bf16>, dim3((int)blocks), dim3(threads), 0, stream, (const bf16*)x, (bf16*)out, (int64_t)total);
     return MIE_ERR_BAD_ARG;
 }
 

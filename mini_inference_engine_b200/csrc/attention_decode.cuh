@@ -20,7 +20,7 @@ struct DecodeParams {
     bf16* out;
     float* out32;            // not null: the output goes here as float32 instead (a caller that subtracts attention outputs)
     float* part_o; float* part_lse; int* counters;      // scratch (splits > 1)
-    int num_heads, num_kv_heads, page_size, page_shift, window, splits, chunks;
+    int num_heads, num_kv_heads, page_size, page_shift, window, keep, splits, chunks;
     int stages;              // tiles in flight per block (2, 3 or 4)
     int min_part_tiles;      // scratch merge: a row is cut into no more parts than it has this many tiles for (0: always `splits`)
     int cluster;             // 1: the splits of a (row, kv head, chunk) are a thread-block cluster and merge through shared memory
@@ -112,7 +112,8 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // this block's part of the context: the range [lo, ctx) cut into `splits` parts of whole tiles
     const int first_key = mask_first_key(ctx - 1, p.window);      // sliding window, or the start of the query's block of positions
     const int lo = first_key & ~(DEC_TILE - 1);
-    const int tiles_total = (ctx - lo + DEC_TILE - 1) / DEC_TILE;
+    const int kept = mask_kept_tiles(p.keep, lo, DEC_TILE);       // tiles of kept keys in front of the window's
+    const int tiles_total = kept + (ctx - lo + DEC_TILE - 1) / DEC_TILE;
     // The grid is laid out for the longest context the launch may meet; a row is cut into as many parts as
     // its own length pays for (scratch merge only: the blocks of a cluster all take part in its barriers).
     // The parts beyond that leave at once, and a row that stays whole writes its output directly.
@@ -125,9 +126,12 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // more, so that no part waits at the merge for one that walked twice as many as it needed to
     const int tiles_base = tiles_total / eff, tiles_more = tiles_total - tiles_base * eff;
     const int tiles_mine = tiles_base + (split < tiles_more ? 1 : 0);
-    const int kbeg = lo + (split * tiles_base + min(split, tiles_more)) * DEC_TILE;
-    const int kend = min(ctx, kbeg + tiles_mine * DEC_TILE);
-    const int ntiles = kend > kbeg ? (kend - kbeg + DEC_TILE - 1) / DEC_TILE : 0;
+    const int tile0 = split * tiles_base + min(split, tiles_more);   // this part's first tile; it has ntiles of them
+    const int ntiles = tiles_mine;
+    auto tile_key = [&](int t) {                                   // where the part's tile t starts
+        const int g = tile0 + t;
+        return g < kept ? g * DEC_TILE : lo + (g - kept) * DEC_TILE;
+    };
 
     float o[NBLK][4];
 #pragma unroll
@@ -148,7 +152,7 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         }
         // A copy brings whole pages; rows of a tile that no page of this part covers keep what the shared
         // memory held.  Their scores are masked, but 0 * NaN is NaN: they must be finite.
-        if ((kend - kbeg) & (DEC_TILE - 1))
+        if (ntiles > 0 && tile_key(ntiles - 1) + DEC_TILE > ctx)
             for (uint32_t i = threadIdx.x * 16; i < (uint32_t)NSTAGE * 2 * KV_TILE_BYTES; i += DEC_WARPS * 32 * 16)
                 *reinterpret_cast<uint4*>(tma_tiles + i) = make_uint4(0, 0, 0, 0);
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // barriers and zeros before the TMA unit touches them
@@ -157,25 +161,35 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // The page ids of this block's part go to shared memory first: a lookup in global memory inside the
     // tile loop would put a memory round trip in front of every tile's copies.
     const int* table = p.block_tables + (int64_t)row * p.table_stride;
-    const int first_page = kbeg >> p.page_shift;
-    const int n_pages = ntiles > 0 ? ((kend - 1) >> p.page_shift) - first_page + 1 : 0;
+    // (A part may hold kept tiles and tiles of the window: the pages of its kept tiles come first in the list.  Entry i is
+    // the table's entry i + kept_page0 or i + page0.)
+    const int kept_mine = max(0, min(kept - tile0, ntiles));
+    const int kept_page0 = (tile0 * DEC_TILE) >> p.page_shift;
+    const int kept_pages = kept_mine > 0 ? (((tile0 + kept_mine) * DEC_TILE - 1) >> p.page_shift) - kept_page0 + 1 : 0;
+    const int rest = ntiles - kept_mine, first_page = rest > 0 ? tile_key(kept_mine) >> p.page_shift : 0, page0 = first_page - kept_pages;
+    const int n_pages = kept_pages + (rest > 0 ? ((min(ctx, tile_key(ntiles - 1) + DEC_TILE) - 1) >> p.page_shift) - first_page + 1 : 0);
     const int64_t page_limit = p.check_pages > 0 ? p.check_pages : ((int64_t)1 << 40);
-    for (int i = threadIdx.x; i < min(n_pages, DEC_PAGE_SLOTS); i += DEC_WARPS * 32)
-        s_pages[i] = checked_page(table[first_page + i], page_limit, p.report, MIE_K_ATTENTION_DECODE, first_page + i);
+    for (int i = threadIdx.x; i < min(n_pages, DEC_PAGE_SLOTS); i += DEC_WARPS * 32) {
+        const int e = i + (i < kept_pages ? kept_page0 : page0);
+        s_pages[i] = checked_page(table[e], page_limit, p.report, MIE_K_ATTENTION_DECODE, e);
+    }
+    auto page_at = [&](int key, int base) {                        // base: kept_page0 for a kept tile's key, else page0
+        const int e = key >> p.page_shift, pi = e - base;
+        return pi < DEC_PAGE_SLOTS ? s_pages[pi] : checked_page(table[e], page_limit, p.report, MIE_K_ATTENTION_DECODE, e);
+    };
     __syncthreads();
     constexpr int CHUNKS_PER_ROW = D / 8;                          // 16-byte pieces per key
     const int rows_per_copy = min(p.page_size, DEC_TILE);          // TMA: one copy = one page (or a 64-row piece of it)
     auto load_tile = [&](int t, int stage) {
-        const int k0 = kbeg + t * DEC_TILE;
+        const int k0 = tile_key(t), base = t < kept_mine ? kept_page0 : page0;
         if (TMA) {
             if (warp == 0) {                                       // lane c copies page c of the tile, keys and values
-                const int copies = (min(DEC_TILE, kend - k0) + rows_per_copy - 1) / rows_per_copy;
+                const int copies = (min(DEC_TILE, ctx - k0) + rows_per_copy - 1) / rows_per_copy;
                 if (lane == 0) mbar_expect_tx(&full_bar[stage], (uint32_t)copies * rows_per_copy * 128u * PARTS * 2u);
                 __syncwarp();
                 if (lane < copies) {
                     const int key = k0 + lane * rows_per_copy;
-                    const int pi = (key >> p.page_shift) - first_page;
-                    const int page = pi < DEC_PAGE_SLOTS ? s_pages[pi] : checked_page(table[first_page + pi], page_limit, p.report, MIE_K_ATTENTION_DECODE, first_page + pi);
+                    const int page = page_at(key, base);
                     const int src_row = (page * p.num_kv_heads + kvh) * p.page_size + (key & (p.page_size - 1));
                     unsigned char* kd = tma_tiles + (size_t)stage * 2 * KV_TILE_BYTES + (size_t)lane * rows_per_copy * 128;
 #pragma unroll
@@ -192,13 +206,12 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         for (int idx = threadIdx.x; idx < DEC_TILE * CHUNKS_PER_ROW; idx += DEC_WARPS * 32) {
             const int r = idx / CHUNKS_PER_ROW, c = (idx - r * CHUNKS_PER_ROW) * 8;
             const int key = k0 + r;
-            if (key < kend) {
-                const int pi = (key >> p.page_shift) - first_page;
-                const int page = pi < DEC_PAGE_SLOTS ? s_pages[pi] : checked_page(table[first_page + pi], page_limit, p.report, MIE_K_ATTENTION_DECODE, first_page + pi);
+            if (key < ctx) {
+                const int page = page_at(key, base);
                 const int64_t src = (((int64_t)page * p.num_kv_heads + kvh) * p.page_size + (key & (p.page_size - 1))) * D + c;
                 cp_async16(kd + r * DP + c, p.k_cache + src);
                 cp_async16(vd + r * DP + c, p.v_cache + src);
-            } else {                                               // beyond the part: zeros, so that 0 * v stays 0
+            } else {                                               // beyond the context: zeros, so that 0 * v stays 0
                 *reinterpret_cast<uint4*>(kd + r * DP + c) = make_uint4(0, 0, 0, 0);
                 *reinterpret_cast<uint4*>(vd + r * DP + c) = make_uint4(0, 0, 0, 0);
             }
@@ -263,15 +276,14 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             cp_async_wait<NSTAGE - 1>();                           // tile t has landed; NSTAGE - 1 younger ones may be in flight
             __syncthreads();
         }
-        if ((rotate || t < NSTAGE - 1) && newest >= kbeg + t * DEC_TILE && newest < min(kend, kbeg + (t + 1) * DEC_TILE)) {
+        if ((rotate || t < NSTAGE - 1) && newest >= tile_key(t) && newest < tile_key(t) + DEC_TILE) {
             // The newest row.  Without rotation here: the tile was copied before the wait and the row may be stale, so it
             // is fetched again (L2, not L1).  With rotation here: the cache does not hold it yet -- this block makes it
             // from the row's q|k|v activation, uses it and writes it into the cache.
             if (threadIdx.x < 2 * CHUNKS_PER_ROW) {
                 const int which = threadIdx.x / CHUNKS_PER_ROW, c = (threadIdx.x - which * CHUNKS_PER_ROW) * 8;
-                const int r = newest - (kbeg + t * DEC_TILE);
-                const int pi = (newest >> p.page_shift) - first_page;
-                const int page = pi < DEC_PAGE_SLOTS ? s_pages[pi] : checked_page(table[first_page + pi], page_limit, p.report, MIE_K_ATTENTION_DECODE, first_page + pi);
+                const int r = newest - tile_key(t);
+                const int page = page_at(newest, page0);           // the newest position lies in the window's last tile, never in a kept one
                 const int64_t src = (((int64_t)page * p.num_kv_heads + kvh) * p.page_size + (newest & (p.page_size - 1))) * D + c;
                 uint4 v;
                 if (rotate) {
@@ -296,8 +308,8 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         const bf16* kt = k_s + stage * DEC_TILE * DP + warp * 16 * DP;
         const bf16* vt = v_s + stage * DEC_TILE * DP + warp * 16 * DP;
         const unsigned char* kt_tma = tma_tiles + (size_t)stage * 2 * KV_TILE_BYTES;   // keys of the stage; values KV_TILE_BYTES behind
-        const int key0 = kbeg + t * DEC_TILE + warp * 16;
-        if (key0 < kend) {                                          // warp-uniform
+        const int key0 = tile_key(t) + warp * 16;
+        if (key0 < ctx) {                                          // warp-uniform
             float s[2][4];
 #pragma unroll
             for (int n = 0; n < 2; ++n) { s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f; }
@@ -312,7 +324,7 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             }
             // mask, scale to base 2, running max
             float mx[2] = {-INFINITY, -INFINITY};
-            const bool whole = key0 + 16 <= kend && key0 >= first_key;   // no key of the warp's 16 needs a mask (warp-uniform)
+            const bool whole = key0 + 16 <= ctx && key0 >= first_key;   // no key of the warp's 16 needs a mask (warp-uniform)
 #pragma unroll
             for (int n = 0; n < 2; ++n)
 #pragma unroll
@@ -325,7 +337,7 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                     }
                     if (!whole) {
                         const int key = key0 + n * 8 + tq * 2 + (i & 1);
-                        if (!(key < kend && key >= first_key)) v = -INFINITY;
+                        if (!(key < ctx && (key >= first_key || key < p.keep))) v = -INFINITY;
                     }
                     s[n][i] = v;
                     mx[i >> 1] = fmaxf(mx[i >> 1], v);
@@ -590,7 +602,7 @@ static int decode_attention_launch(const void* q, int64_t q_stride, const void* 
                                    cudaStream_t stream, int stages = 0, int64_t num_pages = 0,
                                    int64_t check_pages = 0, int* report = nullptr, int min_part_tiles = 0,
                                    const float* cos_t = nullptr, const float* sin_t = nullptr, int max_pos = 0, bool out_f32 = false,
-                                   const ScoreMods* mods = nullptr) {
+                                   const ScoreMods* mods = nullptr, int keep = 0) {
     if (num_rows <= 0) return 0;
     if (head_dim < 16 || head_dim > DEC_MAX_D || head_dim % 16) return MIE_ERR_BAD_ARG;
     if (num_kv_heads <= 0 || num_heads % num_kv_heads) return MIE_ERR_BAD_ARG;
@@ -608,7 +620,7 @@ static int decode_attention_launch(const void* q, int64_t q_stride, const void* 
     p.num_heads = num_heads; p.num_kv_heads = num_kv_heads; p.page_size = page_size;
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
-    p.window = window; p.splits = splits; p.cluster = cluster ? 1 : 0;
+    p.window = window; p.keep = keep > 0 ? keep : 0; p.splits = splits; p.cluster = cluster ? 1 : 0;
     p.stages = stages > 0 ? stages : 4;
     p.min_part_tiles = min_part_tiles > 0 ? min_part_tiles : 0;
     const int G = num_heads / num_kv_heads;

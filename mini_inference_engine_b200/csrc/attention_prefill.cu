@@ -10,7 +10,7 @@
 //   grid.x = query tiles over all rows (64 queries each, longest-running tiles first),
 //   grid.y = query heads.  4 warps, 16 query rows each (mma.sync m16n8k16, bfloat16 in, float32
 //   accumulate).  Keys and values come in tiles of 64 positions through cp.async, two stages.
-//   S = Q K^T for the warp's 16 rows x 64 keys, masked by position (j <= p, j > p - window),
+//   S = Q K^T for the warp's 16 rows x 64 keys, masked by position (j <= p, j > p - window or j < keep),
 //   online softmax in base 2 with float32 max / sum, P rounded to bfloat16, O += P V.
 #include "mma_common.cuh"
 #include "range_check.cuh"
@@ -28,7 +28,7 @@ struct PrefillParams {
     const int* row_q_start; const int* row_q_len; const int* row_ctx_len; int num_rows;
     bf16* out;
     float* out32;      // not null: the output goes here as float32 instead
-    int num_heads, num_kv_heads, page_size, page_shift, window, min_q_len;
+    int num_heads, num_kv_heads, page_size, page_shift, window, keep, min_q_len;
     float scale_log2e;
     int64_t check_pages;     // pages in each cache, for the range check of block-table entries
     int* report;             // range report (range_check.cuh)
@@ -75,7 +75,9 @@ prefill_attention_kernel(const PrefillParams p) {
     const int k_hi = pos0 + nq;                                     // one past the last key any query reads
     const int k_lo = mask_first_key(pos0, p.window);
     const int kbeg = k_lo & ~(PRE_BN - 1);
-    const int ntiles = (k_hi - kbeg + PRE_BN - 1) / PRE_BN;
+    const int kept = mask_kept_tiles(p.keep, kbeg, PRE_BN);         // tiles of kept keys in front of the window's
+    const int ntiles = kept + (k_hi - kbeg + PRE_BN - 1) / PRE_BN;
+    auto tile_key = [&](int t) { return t < kept ? t * PRE_BN : kbeg + (t - kept) * PRE_BN; };
 
     // this warp's 16 queries; thread rows r0 = quad and r1 = quad + 8
     const int wq = warp * 16;
@@ -104,21 +106,26 @@ prefill_attention_kernel(const PrefillParams p) {
     // memory round trip in front of every tile's copies
     const int* table = p.block_tables + (int64_t)row * p.table_stride;
     const int first_page = kbeg >> p.page_shift;
-    const int n_pages = ((k_hi - 1) >> p.page_shift) - first_page + 1;
-    for (int i = threadIdx.x; i < min(n_pages, PRE_PAGE_SLOTS); i += PRE_WARPS * 32)
-        s_pages[i] = checked_page(table[first_page + i], p.check_pages, p.report, MIE_K_ATTENTION_PREFILL, first_page + i);
+    // the pages of the kept tiles first, then those from kbeg on; entry i of the list is the table's entry i or i + skip
+    const int kept_pages = kept > 0 ? ((kept * PRE_BN - 1) >> p.page_shift) + 1 : 0;
+    const int skip = first_page - kept_pages;
+    const int n_pages = kept_pages + ((k_hi - 1) >> p.page_shift) - first_page + 1;
+    for (int i = threadIdx.x; i < min(n_pages, PRE_PAGE_SLOTS); i += PRE_WARPS * 32) {
+        const int e = i < kept_pages ? i : i + skip;
+        s_pages[i] = checked_page(table[e], p.check_pages, p.report, MIE_K_ATTENTION_PREFILL, e);
+    }
     __syncthreads();
     constexpr int CHUNKS_PER_ROW = D / 8;
     auto load_tile = [&](int t, int stage) {
-        const int k0 = kbeg + t * PRE_BN;
+        const int k0 = tile_key(t), page0 = t < kept ? 0 : skip;      // the page list's entry is the table's less page0
         bf16* kd = k_s + stage * PRE_BN * DP;
         bf16* vd = v_s + stage * PRE_BN * DP;
         for (int idx = threadIdx.x; idx < PRE_BN * CHUNKS_PER_ROW; idx += PRE_WARPS * 32) {
             const int r = idx / CHUNKS_PER_ROW, c = (idx - r * CHUNKS_PER_ROW) * 8;
             const int key = k0 + r;
-            if (key >= k_lo && key < k_hi) {
-                const int pi = (key >> p.page_shift) - first_page;
-                const int page = pi < PRE_PAGE_SLOTS ? s_pages[pi] : checked_page(table[first_page + pi], p.check_pages, p.report, MIE_K_ATTENTION_PREFILL, first_page + pi);
+            if ((key >= k_lo || key < p.keep) && key < k_hi) {
+                const int e = key >> p.page_shift, pi = e - page0;
+                const int page = pi < PRE_PAGE_SLOTS ? s_pages[pi] : checked_page(table[e], p.check_pages, p.report, MIE_K_ATTENTION_PREFILL, e);
                 const int64_t src = (((int64_t)page * p.num_kv_heads + kvh) * p.page_size + (key & (p.page_size - 1))) * D + c;
                 cp_async16(kd + r * DP + c, p.k_cache + src);
                 cp_async16(vd + r * DP + c, p.v_cache + src);
@@ -137,7 +144,7 @@ prefill_attention_kernel(const PrefillParams p) {
         cp_async_commit();
         cp_async_wait<1>();
         __syncthreads();
-        const int key0 = kbeg + t * PRE_BN;
+        const int key0 = tile_key(t);
         // a warp whose last query sits before this tile has nothing to read in it
         if (warp_has_rows && key0 <= pos0 + min(wq + 15, nq - 1)) {
             const bf16* kt = k_s + stage * PRE_BN * DP;
@@ -170,7 +177,7 @@ prefill_attention_kernel(const PrefillParams p) {
                     if (need_mask) {
                         const int key = key0 + n * 8 + tq * 2 + (i & 1);
                         const int qp = qpos[i >> 1];
-                        const bool ok = key <= qp && key >= mask_first_key(qp, p.window);
+                        const bool ok = mask_reads(qp, key, p.window, p.keep);
                         v = ok ? v : -INFINITY;
                     }
                     s[n][i] = v;
@@ -266,7 +273,7 @@ extern "C" int mie_prefill_attention(const void* q, int64_t q_stride, const void
                                      const int* block_tables, int table_stride, const int* row_q_start,
                                      const int* row_q_len, const int* row_ctx_len, int num_rows, int num_tokens,
                                      void* out, int num_heads, int num_kv_heads, int head_dim, int page_size,
-                                     float scale, int window, int min_q_len, long long num_pages, int work_rows,
+                                     float scale, int window, int keep, int min_q_len, long long num_pages, int work_rows,
                                      int work_tokens, int out_f32, float softcap, const float* sink, const float* dist_bias,
                                      int dist_len, cudaStream_t stream) {
     if (num_rows <= 0 || num_tokens <= 0) return 0;
@@ -284,7 +291,7 @@ extern "C" int mie_prefill_attention(const void* q, int64_t q_stride, const void
     p.num_heads = num_heads; p.num_kv_heads = num_kv_heads; p.page_size = page_size;
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
-    p.window = window; p.min_q_len = min_q_len;
+    p.window = window; p.keep = keep > 0 ? keep : 0; p.min_q_len = min_q_len;
     p.scale_log2e = scale * 1.4426950408889634f;
     if (dist_bias && dist_len <= 0) return MIE_ERR_BAD_ARG;
     p.scale = scale;

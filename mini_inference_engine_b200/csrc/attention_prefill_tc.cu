@@ -8,7 +8,7 @@
 //               cache one page per copy through the request's block table.  S is 128 x 128 float32 in
 //               TMEM: one query row per TMEM lane.
 //   softmax     four warps, one thread per query row: the thread reads its row of S out of TMEM
-//               (tcgen05.ld), masks by position (key <= query, key > query - window), keeps a running
+//               (tcgen05.ld), masks by position (key <= query, key > query - window or key < keep), keeps a running
 //               max and sum in base 2, and writes P, rounded to bfloat16, back into TMEM (tcgen05.st).
 //               No shuffles: a row never leaves its thread.
 //   O += P V    P is the A operand straight out of TMEM; V [128 keys x D] sits in shared memory as TMA
@@ -45,7 +45,7 @@ struct FaParams {
     bf16* out;
     float* out32;      // not null: the output goes here as float32 instead
     int* error;
-    int num_heads, num_kv_heads, page_size, page_shift, window, min_q_len;
+    int num_heads, num_kv_heads, page_size, page_shift, window, keep, min_q_len;
     int pair;                // 1: a block takes two query tiles of a row (see the kernel), 0: one
     float scale_log2e;
     int64_t check_pages;     // pages in each cache, for the range check of block-table entries
@@ -192,7 +192,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
         const int kvh = head / (p.num_heads / p.num_kv_heads);
         const int nsub = s_nsub;
         // the geometry of query tile u: first query's position, rows, key range in tiles of FA_BN keys
-        struct Sub { int q0, pos0, nq, k_hi, k_lo, kbeg, ntiles; };
+        struct Sub { int q0, pos0, nq, k_hi, k_lo, kbeg, kept, ntiles; };
         Sub sb[2];
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
@@ -203,7 +203,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
             g.k_hi = g.pos0 + g.nq;                              // one past the last key any query here reads
             g.k_lo = mask_first_key(g.pos0, p.window);
             g.kbeg = g.k_lo & ~(FA_BN - 1);
-            g.ntiles = u < nsub ? (g.k_hi - g.kbeg + FA_BN - 1) / FA_BN : 0;
+            g.kept = mask_kept_tiles(p.keep, g.kbeg, FA_BN);     // tiles of kept keys in front of the window's
+            g.ntiles = u < nsub ? g.kept + (g.k_hi - g.kbeg + FA_BN - 1) / FA_BN : 0;
         }
         const int nA = sb[0].ntiles, G = nA + sb[1].ntiles;      // key tiles of the first query tile, and of both
         // Key tiles are counted through both query tiles (g = 0 .. G-1): stages and barrier phases go on
@@ -223,7 +224,10 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                         tma_load_2d(tiles + u * Q_BYTES + part * SUB_BYTES, &map_q, &q_full[u], head * D + part * 64, q_start + sb[u].q0);
                 }
             }
-            auto key0_of = [&](int g) { return g < nA ? sb[0].kbeg + g * FA_BN : sb[1].kbeg + (g - nA) * FA_BN; };
+            auto key0_of = [&](int g) {
+                const int t = g < nA ? g : g - nA, kept = g < nA ? sb[0].kept : sb[1].kept;
+                return t < kept ? t * FA_BN : (g < nA ? sb[0].kbeg : sb[1].kbeg) + (t - kept) * FA_BN;
+            };
             auto copies_of = [&](int g) {
                 const int key0 = key0_of(g), hi = g < nA ? sb[0].k_hi : sb[1].k_hi;
                 return (min(key0 + FA_BN, hi) - key0 + rows_per_copy - 1) / rows_per_copy;
@@ -344,7 +348,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
             const uint32_t lane_addr = tmem_base + ((uint32_t)(q * 32) << 16);
             bool ok = true;
             for (int u = 0; u < nsub && ok; ++u) {                 // one query tile after the other
-                const int q0 = sb[u].q0, pos0 = sb[u].pos0, nq = sb[u].nq, k_lo = sb[u].k_lo, kbeg = sb[u].kbeg, ntiles = sb[u].ntiles;
+                const int q0 = sb[u].q0, pos0 = sb[u].pos0, nq = sb[u].nq, k_lo = sb[u].k_lo, kbeg = sb[u].kbeg, kept = sb[u].kept, ntiles = sb[u].ntiles;
                 const int g0 = u ? nA : 0;                             // key tiles counted through both query tiles
                 const int qpos = pos0 + r;
                 float m_run = -INFINITY, l_run = 0.f;
@@ -365,7 +369,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                     ok = __all_sync(0xffffffffu, mbar_wait(&s_full, g & 1, abort_p));     // the warp goes on or gives up as one
                     if (!ok) break;
                     tc_fence_after();
-                    const int key0 = kbeg + t * FA_BN;
+                    const int key0 = t < kept ? t * FA_BN : kbeg + (t - kept) * FA_BN;
                     // masks are needed only where the tile touches the diagonal, the window's edge or the range's start
                     const bool need_mask = key0 + FA_BN - 1 > pos0 || key0 < k_lo || (p.window != 0 && key0 < mask_first_key(pos0 + FA_BM - 1, p.window));
                     // The row of S comes out of TMEM in four chunks of 32 columns; the load of the next chunk is
@@ -385,7 +389,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                         tmem_ld_wait(cb);
                         body(3, cb);
                     };
-                    auto masked = [&](int key) { return !(key <= qpos && key >= mask_first_key(qpos, p.window)); };
+                    auto masked = [&](int key) { return !mask_reads(qpos, key, p.window, p.keep); };
                     // Reference point of the exponent.  Reading S once per tile is what matters here (TMEM
                     // loads are the slowest part of the step), so the running max is not recomputed up front:
                     // P is formed against the running max as it stands, the row's true max is found on the
@@ -950,7 +954,7 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
                                         int64_t num_pages, const int* block_tables, int table_stride, const int* row_q_start,
                                         const int* row_q_len, const int* row_ctx_len, int num_rows, int num_tokens, void* out,
                                         int num_heads, int num_kv_heads, int head_dim, int page_size, float scale, int window,
-                                        int min_q_len, int work_rows, int work_tokens, int out_f32, float softcap, const float* sink,
+                                        int keep, int min_q_len, int work_rows, int work_tokens, int out_f32, float softcap, const float* sink,
                                         const float* dist_bias, int dist_len, cudaStream_t stream) {
     if (num_rows <= 0 || num_tokens <= 0) return 0;
     if (work_rows <= 0 || work_tokens <= 0 || work_rows > num_rows || work_tokens > num_tokens) { work_rows = num_rows; work_tokens = num_tokens; }
@@ -968,7 +972,7 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
     p.num_heads = num_heads; p.num_kv_heads = num_kv_heads; p.page_size = page_size;
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
-    p.window = window; p.min_q_len = min_q_len; p.pair = 0;
+    p.window = window; p.keep = keep > 0 ? keep : 0; p.min_q_len = min_q_len; p.pair = 0;
     p.scale_log2e = scale * 1.4426950408889634f;
     p.scale = scale;
     p.mods = ScoreMods{softcap, sink, dist_bias, dist_len};
@@ -986,7 +990,7 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
                                  : launch_fa<DD, 3>(mq, mk, mv, p, work_tokens, work_rows, stream))
     if (mods) return head_dim == 64 ? FA_MODS(64) : FA_MODS(128);
 #undef FA_MODS
-    if (head_dim == 64 && !sink) {        // (the kernel with two query tiles side by side has no sink)
+    if (head_dim == 64 && !sink && p.keep == 0) {        // (the kernel with two query tiles side by side has no sink and no kept keys)
         // two query tiles side by side once there are three pairs for every SM (measured, 32 heads, one tile a block
         // against two side by side: 2,048 tokens 45.1 against 48.5 us, 4,096 tokens 143.7 against 142.4 us, 8,192 tokens
         // 496 against 462 us); below that the one-tile blocks, two on an SM, spread a launch over more SMs

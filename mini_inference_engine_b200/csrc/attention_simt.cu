@@ -4,7 +4,7 @@
 //
 // A batch row is a request: q_len new tokens whose keys and values were already written to the
 // cache, ctx_len = tokens in the cache including them.  Query i of the row sits at position
-// p = ctx_len - q_len + i and reads keys j <= p (from mask_first_key(p, window) on: a sliding window or its own block of positions) through the
+// p = ctx_len - q_len + i and reads keys j <= p (from mask_first_key(p, window) on: a sliding window or its own block of positions; and the first `keep` keys) through the
 // row's block table.  Query head h reads kv head h / (H / H_kv).  Scores, softmax and the
 // accumulator are float32; online softmax over tiles of 32 keys.  A score may be capped, take a bias by distance and share
 // the softmax with a sink (ScoreMods, common.cuh).
@@ -53,7 +53,7 @@ paged_attention_kernel(const T* __restrict__ q, int64_t q_stride, const T* __res
                        const int* __restrict__ row_q_len, const int* __restrict__ row_ctx_len,
                        int num_rows, TO* __restrict__ out, int num_heads, int num_kv_heads,
                        int head_dim, int page_size, int page_shift, float scale, int window,
-                       int QT, int HG, int min_q_len, int64_t num_pages, int* report, const ScoreMods mods) {
+                       int keep, int QT, int HG, int min_q_len, int64_t num_pages, int* report, const ScoreMods mods) {
     extern __shared__ __align__(16) float smem[];
     __shared__ int s_row, s_q0;
     const int D = head_dim, DP = head_dim + 4;
@@ -109,13 +109,15 @@ paged_attention_kernel(const T* __restrict__ q, int64_t q_stride, const T* __res
     const int vecs_per_row = D / Vec<T>::N;
     const int* table = block_tables + (int64_t)r * table_stride;
 
-    for (int k0 = k_lo & ~(ATT_KEYS - 1); k0 < k_hi; k0 += ATT_KEYS) {
+    const int kbeg = k_lo & ~(ATT_KEYS - 1), kept = mask_kept_tiles(keep, kbeg, ATT_KEYS);
+    for (int t = 0; t < kept || kbeg + (t - kept) * ATT_KEYS < k_hi; ++t) {
+        const int k0 = t < kept ? t * ATT_KEYS : kbeg + (t - kept) * ATT_KEYS;
         __syncthreads();                     // the previous tile (and q_s on the first pass) is done with
         for (int idx = threadIdx.x; idx < ATT_KEYS * vecs_per_row; idx += blockDim.x) {
             const int jj = idx / vecs_per_row, c = (idx - jj * vecs_per_row) * Vec<T>::N;
             const int key = k0 + jj;
             float kf[Vec<T>::N], vf[Vec<T>::N];
-            if (key >= k_lo && key < k_hi) {
+            if ((key >= k_lo || key < keep) && key < k_hi) {
                 const int page = checked_page(table[key >> page_shift], num_pages, report, MIE_K_ATTENTION_SIMT, key >> page_shift);
                 const int off = key & (page_size - 1);
                 const int64_t src = (((int64_t)page * num_kv_heads + kvh) * page_size + off) * D + c;
@@ -131,7 +133,7 @@ paged_attention_kernel(const T* __restrict__ q, int64_t q_stride, const T* __res
         __syncthreads();
         if (active) {
             const int key = k0 + lane;
-            const bool valid = key <= pos_q && key >= mask_first_key(pos_q, window);
+            const bool valid = mask_reads(pos_q, key, window, keep);
             float s = 0.f;
             const float4* kr = reinterpret_cast<const float4*>(k_s + lane * DP);
             const float4* qr = reinterpret_cast<const float4*>(q_s + warp * D);
@@ -182,7 +184,7 @@ extern "C" int mie_paged_attention(const void* q, int64_t q_stride, const void* 
                                    const int* block_tables, int table_stride, const int* row_q_start,
                                    const int* row_q_len, const int* row_ctx_len, int num_rows,
                                    int num_tokens, void* out, int act_tag, int num_heads, int num_kv_heads,
-                                   int head_dim, int page_size, float scale, int window, int min_q_len,
+                                   int head_dim, int page_size, float scale, int window, int keep, int min_q_len,
                                    long long num_pages, int out_f32, float softcap, const float* sink, const float* dist_bias,
                                    int dist_len, cudaStream_t stream) {
     if (num_rows <= 0 || num_tokens <= 0) return 0;
@@ -206,21 +208,21 @@ extern "C" int mie_paged_attention(const void* q, int64_t q_stride, const void* 
         return launch_kernel(paged_attention_kernel<float, float>, grid, dim3(ATT_WARPS * 32), smem, stream,
             (const float*)q, q_stride, (const float*)k_cache, (const float*)v_cache, block_tables, table_stride,
             row_q_start, row_q_len, row_ctx_len, num_rows, (float*)out, num_heads, num_kv_heads, head_dim,
-            page_size, page_shift, scale, window, QT, HG, min_q_len, (int64_t)num_pages, g_range_report, mods);
+            page_size, page_shift, scale, window, keep, QT, HG, min_q_len, (int64_t)num_pages, g_range_report, mods);
     } else if (act_tag == MIE_BF16 && out_f32) {             // bfloat16 operands, the output left in float32
         e = cudaFuncSetAttribute(paged_attention_kernel<bf16, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         return launch_kernel(paged_attention_kernel<bf16, float>, grid, dim3(ATT_WARPS * 32), smem, stream,
             (const bf16*)q, q_stride, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, table_stride,
             row_q_start, row_q_len, row_ctx_len, num_rows, (float*)out, num_heads, num_kv_heads, head_dim,
-            page_size, page_shift, scale, window, QT, HG, min_q_len, (int64_t)num_pages, g_range_report, mods);
+            page_size, page_shift, scale, window, keep, QT, HG, min_q_len, (int64_t)num_pages, g_range_report, mods);
     } else if (act_tag == MIE_BF16) {
         e = cudaFuncSetAttribute(paged_attention_kernel<bf16, bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         return launch_kernel(paged_attention_kernel<bf16, bf16>, grid, dim3(ATT_WARPS * 32), smem, stream,
             (const bf16*)q, q_stride, (const bf16*)k_cache, (const bf16*)v_cache, block_tables, table_stride,
             row_q_start, row_q_len, row_ctx_len, num_rows, (bf16*)out, num_heads, num_kv_heads, head_dim,
-            page_size, page_shift, scale, window, QT, HG, min_q_len, (int64_t)num_pages, g_range_report, mods);
+            page_size, page_shift, scale, window, keep, QT, HG, min_q_len, (int64_t)num_pages, g_range_report, mods);
     }
     return MIE_ERR_BAD_ARG;
 }

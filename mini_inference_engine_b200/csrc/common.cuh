@@ -25,6 +25,18 @@ __host__ __device__ __forceinline__ int mask_first_key(int pos, int window) {
     if (window < 0) return pos - pos % (-window);
     return 0;
 }
+// A window or a block may also keep the first `keep` keys of the sequence in sight (at their true positions): a query reads key j
+// when j is not later than itself and lies in the window (or block) or among the kept ones.  keep 0: none.
+__host__ __device__ __forceinline__ bool mask_reads(int pos, int key, int window, int keep) {
+    return key <= pos && (key >= mask_first_key(pos, window) || key < keep);
+}
+// A kernel that walks keys in tiles of `tile` from `kbeg` on (a multiple of `tile`, at or before the first key of the window) walks
+// the kept keys' tiles first: so many of them lie before kbeg.  Tile t of the walk starts at key t * tile for t below this
+// number and at kbeg + (t - this number) * tile from there on.
+__host__ __device__ __forceinline__ int mask_kept_tiles(int keep, int kbeg, int tile) {
+    const int n = (keep + tile - 1) / tile, before = kbeg / tile;
+    return keep <= 0 ? 0 : n < before ? n : before;
+}
 
 // What may happen to an attention score between the scaled product q . k and the softmax, each switched by its field:
 struct ScoreMods {

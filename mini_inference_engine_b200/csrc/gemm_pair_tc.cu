@@ -43,7 +43,7 @@ typedef __nv_bfloat16 bf16;
 struct GpParams {
     void* out;               // [M, N] (or [M, N / 2] with SwiGLU), bfloat16 or float32
     const void* bias;        // [N] or null
-    int bias_tag, out_f32, swiglu;           // swiglu 1: the gated epilogue; 2: an activation on every output (xIELU), y stays N wide
+    int bias_tag, out_f32, swiglu;           // swiglu 1: the gated epilogue; 2, 3: an activation on every output (xIELU; the square of relu), y stays N wide
     float glu_limit, glu_slope, glu_shift;   // the gated epilogue's shape: g' sigmoid(slope g') (u' + shift) with clamps at +-limit (<= 0: none); 0, 1, 0 is SwiGLU
                                              // with swiglu 2: slope = a_p, shift = a_n of a_p z^2 + z / 2 (z > 0), a_n (exp(z) - 1 - z) + z / 2 (z <= 0)
     int M, N, K;
@@ -254,6 +254,10 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
                         v[i] = xielu_epilogue(v[i], p.glu_slope, p.glu_shift);
                     }
                 }
+                if (p.swiglu == 3) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) { const float z = fmaxf(v[i], 0.f); v[i] = z * z; }
+                }
                 if (p.swiglu == 1) {
                     // interleaved rows of w: column 2i the gate, 2i + 1 the value
                     float o[16];
@@ -350,7 +354,7 @@ extern "C" int mie_gemm_pair(const void* x, const void* w, const void* bias, int
                              int K, int swiglu, float glu_limit, float glu_slope, float glu_shift, const GpFuse* fuse,
                              cudaStream_t stream) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;
-    if (K % 8 || N % 8 || (swiglu == 1 && N % 16) || swiglu < 0 || swiglu > 2) return MIE_ERR_BAD_ARG;
+    if (K % 8 || N % 8 || (swiglu == 1 && N % 16) || swiglu < 0 || swiglu > 3) return MIE_ERR_BAD_ARG;
     const bool into_stream = fuse && fuse->res;
     if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | (into_stream ? 0 : reinterpret_cast<uintptr_t>(y))) & 15) return MIE_ERR_BAD_ARG;
     if (!into_stream && (!y || (y_tag != MIE_BF16 && y_tag != MIE_F32))) return MIE_ERR_BAD_ARG;

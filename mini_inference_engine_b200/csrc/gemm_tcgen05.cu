@@ -77,7 +77,7 @@ struct TcParams {
     int M, N, K;             // tokens, output features (rows of W), inner size
     int k_tiles, tiles_per_split, splits, stages;
     int l2_ahead;            // weight k-tiles beyond the ring that the copy warp asks into L2 before the dependency wait
-    int swiglu;              // 1: rows 2i / 2i+1 of W are gate_i / up_i; the output is glu(gate, up), N/2 wide
+    int swiglu;              // 1: rows 2i / 2i+1 of W are gate_i / up_i; the output is glu(gate, up), N/2 wide; 2: every output is max(z, 0)^2
     float glu_limit, glu_slope, glu_shift;   // glu(g, u) = g' sigmoid(slope g') (u' + shift), g' = min(g, limit), u' = clamp(u, +-limit)
                                              // (limit <= 0: no clamp); 0, 1, 0 is SwiGLU
     // Optional fused rotation + cache write for a q|k|v projection (see the header comment): rows of W
@@ -139,6 +139,11 @@ __device__ __forceinline__ float glu_mul(float g, float u, float limit, float sl
     if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
     const float z = limit < 0.f ? slope * g * fmaf(-limit * g, g, 1.0f) : slope * g;      // a negative limit: no clamp, -limit the cubic term (gelu's tanh form)
     return __fdividef(g, 1.0f + __expf(-z)) * (u + shift);
+}
+// an activation on a plain output (swiglu 2)
+__device__ __forceinline__ float plain_act(float z, int swiglu) {
+    const float r = fmaxf(z, 0.f);
+    return swiglu == 2 ? r * r : z;
 }
 #define GLU_OF(g, u) glu_mul(g, u, p.glu_limit, p.glu_slope, p.glu_shift)      // inside a kernel whose parameters are `p`
 
@@ -430,7 +435,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,     // the 128-row ope
 #pragma unroll
                             for (int i = 0; i < 16; ++i) if (n + i < p.N) v[i] += load_tagged(p.bias, n + i, p.bias_tag);
                         }
-                        if (p.swiglu) {
+                        if (p.swiglu == 1) {
                             float h[16];
 #pragma unroll
                             for (int i = 0; i < 8; ++i) h[i] = GLU_OF(v[2 * i], v[2 * i + 1]);
@@ -449,6 +454,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,     // the 128-row ope
                                 *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.out) + (int64_t)m * (p.N / 2) + n / 2) = w;
                             }
                         } else {
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) v[i] = plain_act(v[i], p.swiglu);
                             store_row16<OUT_F32>(p.out, (int64_t)m * p.N, n, p.N, v);
                         }
                     }
@@ -459,12 +466,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,     // the 128-row ope
                     for (int i = 0; i < 16; ++i) {
                         const int t = b0 + c + i;
                         float val = v[i] + b;
-                        if (p.swiglu) {                        // gate on the even lane, up on the odd one
+                        if (p.swiglu == 1) {                        // gate on the even lane, up on the odd one
                             const float other = __shfl_xor_sync(0xffffffffu, val, 1);
                             if (!(lane & 1) && t < p.M && n < p.N)
                                 store_out<OUT_F32>(p.out, (int64_t)t * (p.N / 2) + n / 2, GLU_OF(val, other));
                         } else if (t < p.M && n < p.N) {
-                            store_out<OUT_F32>(p.out, (int64_t)t * p.N + n, val);
+                            store_out<OUT_F32>(p.out, (int64_t)t * p.N + n, plain_act(val, p.swiglu));
                         }
                     }
                 }
@@ -584,11 +591,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,     // the 128-row ope
                     if (j >= tpo) continue;
                     const int t = b0 + tk0 + j;
                     const float val = acc[j] + b;
-                    if (p.swiglu) {                            // gate on the even row, up on the odd one: neighbouring lanes
+                    if (p.swiglu == 1) {                            // gate on the even row, up on the odd one: neighbouring lanes
                         const float other = __shfl_xor_sync(0xffffffffu, val, 1);
                         if (!(r & 1) && t < p.M && live) store_out<OUT_F32>(p.out, (int64_t)t * (p.N / 2) + n / 2, GLU_OF(val, other));
                     } else if (t < p.M && live) {
-                        store_out<OUT_F32>(p.out, (int64_t)t * p.N + n, val);
+                        store_out<OUT_F32>(p.out, (int64_t)t * p.N + n, plain_act(val, p.swiglu));
                     }
                 }
             }
@@ -625,12 +632,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,     // the 128-row ope
 #pragma unroll
                         for (int j = 0; j < 4; ++j) acc[j] += load_tagged(p.bias, n + j, p.bias_tag);
                     }
-                    if (p.swiglu) {
+                    if (p.swiglu == 1) {
                         store_out<OUT_F32>(p.out, (int64_t)m * (p.N / 2) + n / 2, GLU_OF(acc[0], acc[1]));
                         store_out<OUT_F32>(p.out, (int64_t)m * (p.N / 2) + n / 2 + 1, GLU_OF(acc[2], acc[3]));
                     } else {
 #pragma unroll
-                        for (int j = 0; j < 4; ++j) store_out<OUT_F32>(p.out, (int64_t)m * p.N + n + j, acc[j]);
+                        for (int j = 0; j < 4; ++j) store_out<OUT_F32>(p.out, (int64_t)m * p.N + n + j, plain_act(acc[j], p.swiglu));
                     }
                 } else if (p.rope) {
                     const int n = a0 + rr;
@@ -736,12 +743,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,     // the 128-row ope
                     for (int j = 0; j < 4; ++j) {
                         const int t = b0 + c + j;
                         const float val = acc[j] + b;
-                        if (p.swiglu) {                        // gate on the even feature, up on the odd one: neighbouring threads
+                        if (p.swiglu == 1) {                        // gate on the even feature, up on the odd one: neighbouring threads
                             const float other = __shfl_xor_sync(0xffffffffu, val, 1);
                             if (!(rr & 1) && t < p.M && n < p.N)
                                 store_out<OUT_F32>(p.out, (int64_t)t * (p.N / 2) + n / 2, GLU_OF(val, other));
                         } else if (t < p.M && n < p.N) {
-                            store_out<OUT_F32>(p.out, (int64_t)t * p.N + n, val);
+                            store_out<OUT_F32>(p.out, (int64_t)t * p.N + n, plain_act(val, p.swiglu));
                         }
                     }
                 }
@@ -862,7 +869,7 @@ static int gemm_tc_launch(const void* x, const void* w, const void* bias, int bi
                           cudaStream_t stream, const TcFuse* fuse = nullptr, float glu_limit = 0.f, float glu_slope = 1.f,
                           float glu_shift = 0.f) {
     if (M <= 0 || N <= 0) return 0;
-    if (K <= 0 || K % 8 || N % 8 || (swiglu && N % 16)) return MIE_ERR_BAD_ARG;
+    if (K <= 0 || K % 8 || N % 8 || (swiglu == 1 && N % 16)) return MIE_ERR_BAD_ARG;
     if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(y)) & 15) return MIE_ERR_BAD_ARG;
     const bool to_res = fuse && fuse->res;
     if (stages < 2 || stages > TC_MAX_STAGES) return MIE_ERR_BAD_ARG;

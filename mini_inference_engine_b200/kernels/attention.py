@@ -57,10 +57,12 @@ def rotates_in_decode(dtype, head_dim: int, ctx) -> bool:
             and decode_only(ctx))
 
 
-def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, window, rope=None, q_stride=None, mods=None):
+def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, window, rope=None, q_stride=None, mods=None,
+              keep: int = 0):
     """``rope`` = (cos, sin): ``qkv`` is unrotated and the cache rows of the new tokens are unwritten; only
     where ``rotates_in_decode`` holds.  ``window``: None or 0 all earlier keys, w > 0 the last w positions, w < 0 the
-    keys of the query's own block of -w positions.  ``q_stride``: elements between the token rows of ``qkv`` (by
+    keys of the query's own block of -w positions.  ``keep``: beside a window or block, the first ``keep`` keys of the
+    sequence stay in sight.  ``q_stride``: elements between the token rows of ``qkv`` (by
     default rows of a fused q|k|v projection).  ``mods`` (``ops.ScoreMods``): a cap on the scores, a bias by distance, a sink in
     the softmax; every kernel applies them (the tcgen05 kernel for portions in an instance of its own)."""
     if q_stride is None:
@@ -70,10 +72,11 @@ def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, wi
     fast = _backend == "auto" and qkv.dtype == torch.bfloat16 and head_dim <= 128
     window = int(window or 0)
     # the keys a single new token can reach, for the decode kernel's plan: a window or a block of positions bounds them
-    reach = ctx.max_ctx_len if window == 0 else min(ctx.max_ctx_len, abs(window) + 64)
+    keep = int(keep or 0) if window else 0              # (without a window every key is in sight already)
+    reach = ctx.max_ctx_len if window == 0 else min(ctx.max_ctx_len, abs(window) + 64 + -(-keep // 64) * 64)
     if rope is not None:
-        if mods is not None:
-            raise ValueError("rotation inside attention and score modifiers do not go together")
+        if mods is not None or keep:
+            raise ValueError("rotation inside attention does not go together with score modifiers or kept keys")
         if not rotates_in_decode(qkv.dtype, head_dim, ctx):
             raise ValueError("rotation inside attention serves steps of decoding rows only (bfloat16, head sizes "
                              "in steps of 32 up to 128)")
@@ -81,7 +84,7 @@ def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, wi
                                     max_ctx=ctx.max_ctx_len, rope=rope)
     if not fast:
         return ops.paged_attention(*args, ctx.num_tokens, out, num_heads, num_kv_heads, head_dim, cache.page_size,
-                                   scale, window, mods=mods)
+                                   scale, window, mods=mods, keep=keep)
     kinds = _row_kinds(ctx)
     has_decode = kinds is None or kinds[0] > 0
     has_prefill = kinds is None or kinds[1] > 0
@@ -92,7 +95,7 @@ def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, wi
         has_decode, min_q_len = False, 1
     if has_decode:
         ops.decode_attention(*args, out, num_heads, num_kv_heads, head_dim, cache.page_size, scale, window,
-                             max_ctx=reach, mods=mods)
+                             max_ctx=reach, mods=mods, keep=keep)
     if has_prefill:
         # tcgen05 (S and O in tensor memory) for the head sizes it is written for, mma.sync otherwise
         tc = head_dim in (64, 128) and cache.page_size >= 8 and q_stride % 8 == 0 and _prefill_backend == "tcgen05"
@@ -100,5 +103,5 @@ def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, wi
         # the rows that are portions, and their tokens: the launch is laid out for those, not for every decoding row
         work = None if kinds is None else (kinds[1], kinds[2])
         fn(*args, ctx.num_tokens, out, num_heads, num_kv_heads, head_dim, cache.page_size, scale, window,
-           min_q_len=min_q_len, work=work, mods=mods)
+           min_q_len=min_q_len, work=work, mods=mods, keep=keep)
     return out

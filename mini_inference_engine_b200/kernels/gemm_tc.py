@@ -297,11 +297,14 @@ def gemm_residual(x, w: torch.Tensor, res: torch.Tensor, bias=None, norm_weight=
 SWIGLU = (0.0, 1.0, 0.0)       # the gated epilogue's (limit, slope, shift) that make it silu(gate) * up
 
 
-def gemm(x, w: torch.Tensor, out: torch.Tensor, bias=None, swiglu: bool = False, glu=None, **force) -> torch.Tensor:
+def gemm(x, w: torch.Tensor, out: torch.Tensor, bias=None, swiglu: bool = False, glu=None, relu2: bool = False, **force) -> torch.Tensor:
     """out[M, N] = x[M, K] @ w[N, K]^T (+ bias) with bfloat16 operands on tcgen05.  With ``swiglu`` the
     rows of ``w`` are gate/up interleaved and out is [M, N/2] = silu(gate) * up -- or, with ``glu`` =
     (limit, slope, shift), g sigmoid(slope g) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit)
-    (limit <= 0: no clamp).  ``x`` may be a DeferredNorm (sizes must then satisfy ``splits_k``)."""
+    (limit <= 0: no clamp).  ``relu2``: every output is max(z, 0)^2, squared in float32 before it is rounded.  ``x`` may be a
+    DeferredNorm (sizes must then satisfy ``splits_k``)."""
+    if relu2 and (swiglu or isinstance(x, DeferredNorm)):
+        raise GemmTcError("gemm: the activation epilogue goes with a plain product of a plain input")
     glu = tuple(float(v) for v in (glu or SWIGLU))
     deferred = x if isinstance(x, DeferredNorm) else None
     if deferred is not None:
@@ -326,7 +329,7 @@ def gemm(x, w: torch.Tensor, out: torch.Tensor, bias=None, swiglu: bool = False,
     lib = ops.load("gemm_tcgen05")
     rc = lib.mie_gemm_tc(ops._ptr(x), ops._ptr(w), ops._ptr(bias), ops.tag(bias) if bias is not None else 0,
                          ops._ptr(out), ops.tag(out), M, N, K, int(pl["swapped"]), pl["bn"], pl["splits"], pl["stages"],
-                         int(swiglu), ctypes.c_float(glu[0]), ctypes.c_float(glu[1]), ctypes.c_float(glu[2]),
+                         2 if relu2 else int(swiglu), ctypes.c_float(glu[0]), ctypes.c_float(glu[1]), ctypes.c_float(glu[2]),
                          int(pl.get("pdl", pdl_enabled)), ops._stream())
     ops._check(rc, f"gemm_tc M{M} N{N} K{K} {pl}")
     return out
@@ -388,20 +391,21 @@ def pair_supports(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: b
 
 
 def gemm_pair(x, w: torch.Tensor, out: torch.Tensor | None, bias: torch.Tensor | None = None, swiglu: bool = False,
-              res: torch.Tensor | None = None, norm_weight: torch.Tensor | None = None, eps: float = 0.0, glu=None, xielu=None):
+              res: torch.Tensor | None = None, norm_weight: torch.Tensor | None = None, eps: float = 0.0, glu=None, xielu=None, relu2: bool = False):
     """out = x w^T (+ bias), or silu(gate) * value over interleaved rows of ``w`` with ``swiglu``: the product
     for many tokens on pairs of SMs (``csrc/gemm_pair_tc.cu``: 256 x 256 tiles by cta_group::2 MMAs, two
     accumulators in tensor memory, one persistent pair of blocks per two SMs).  ``x`` may be a DeferredNorm (the
     norm in front becomes a row factor on the sums).  With ``res`` (float32 [M, N]) the product is added to it
     in place instead of being written (``out`` is None); with ``norm_weight`` as well, the DeferredNorm for the
     product behind that norm is returned.  ``xielu`` = (a_p, a_n): every output goes through that activation in the
-    epilogue (a_p z^2 + z / 2 for z > 0, a_n (exp(z) - 1 - z) + z / 2 else), in float32 before it is rounded."""
+    epilogue (a_p z^2 + z / 2 for z > 0, a_n (exp(z) - 1 - z) + z / 2 else), in float32 before it is rounded; ``relu2``: through
+    max(z, 0)^2."""
     glu = tuple(float(v) for v in (glu or SWIGLU))        # the gated epilogue's shape, as for ``gemm``
     mode = int(swiglu)
-    if xielu is not None:
-        if swiglu or res is not None:
+    if xielu is not None or relu2:
+        if swiglu or res is not None or (relu2 and xielu is not None):
             raise GemmTcError("gemm_pair: the activation epilogue goes with a plain product")
-        mode, glu = 2, (0.0, float(xielu[0]), float(xielu[1]))
+        mode, glu = (3, SWIGLU) if relu2 else (2, (0.0, float(xielu[0]), float(xielu[1])))
     deferred = x if isinstance(x, DeferredNorm) else None
     xt = deferred.xw if deferred is not None else x
     M, K = xt.shape

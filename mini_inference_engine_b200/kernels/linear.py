@@ -150,6 +150,23 @@ def linear_xielu(x: torch.Tensor, w: torch.Tensor, ap: float, an: float, out_dty
     return ops.xielu(up, torch.empty_like(up), ap, an)
 
 
+def linear_relu2(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """max(x W^T, 0)^2: in the epilogue of the tcgen05 products where they run (a few tokens; prompt-sized steps on pairs of SMs),
+    else the product followed by the activation kernel."""
+    M = x.shape[0]
+    if M and x.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and not isinstance(x, gemm_tc.DeferredNorm):
+        if takes_pair(M, w) and x.is_contiguous():
+            out = torch.empty(M, w.shape[0], dtype=out_dtype, device=w.device)
+            if gemm_tc.pair_supports(x, w, out):
+                return gemm_tc.gemm_pair(x, w, out, relu2=True)
+        if uses_tcgen05(x, w):
+            out = torch.empty(M, w.shape[0], dtype=out_dtype, device=w.device)
+            if gemm_tc.supports(x, w, out):
+                return gemm_tc.gemm(x, w, out, relu2=True)
+    up = linear(x, w, None, out_dtype)
+    return ops.relu2(up, up)
+
+
 def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out_dtype: torch.dtype, glu=None) -> torch.Tensor:
     """silu(x Wg^T) * (x Wu^T) for a weight whose rows alternate gate_i, up_i: fused into the
     tcgen05 product's epilogue where that kernel runs, else the product followed by the SwiGLU kernel.

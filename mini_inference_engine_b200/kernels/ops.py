@@ -216,6 +216,13 @@ def xielu(x: torch.Tensor, out: torch.Tensor, ap: float, an: float) -> torch.Ten
     return out
 
 
+def relu2(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out = max(x, 0)^2 (``out`` may be ``x``)."""
+    _need(x.is_contiguous() and out.is_contiguous() and out.shape == x.shape and out.dtype == x.dtype, "relu2: contiguous tensors of one shape and type")
+    _check(load("activation").mie_relu2(_ptr(x), _ptr(out), tag(x), ctypes.c_longlong(x.numel()), _stream()), "relu2")
+    return out
+
+
 def gelu_gate_rows(g: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, first: int, out: torch.Tensor) -> torch.Tensor:
     """out[t, d] = gelu_tanh(g[t, d]) * table[ids[t], first + d]."""
     T, n = g.shape
@@ -360,10 +367,10 @@ _NO_MODS = ScoreMods()
 def paged_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_tables, row_q_start, row_q_len,
                     row_ctx_len, num_tokens: int, out: torch.Tensor, num_heads: int, num_kv_heads: int,
                     head_dim: int, page_size: int, scale: float, window: int | None = None,
-                    min_q_len: int = 1, mods: ScoreMods | None = None) -> torch.Tensor:
+                    min_q_len: int = 1, mods: ScoreMods | None = None, keep: int = 0) -> torch.Tensor:
     """Causal attention of every new token over its request's pages (CUDA-core kernel, float32 or
     bfloat16).  ``q`` holds [H, D] at the start of each token row of ``q_stride`` elements.  Rows
-    with fewer than ``min_q_len`` new tokens are left alone."""
+    with fewer than ``min_q_len`` new tokens are left alone.  ``keep``: with a window, the first that many keys stay in sight too."""
     _need(head_dim % 16 == 0 and 16 <= head_dim <= 256,
           f"head_dim {head_dim}: this kernel takes multiples of 16 from 16 to 256")
     _need(num_heads % num_kv_heads == 0, "query heads must be a multiple of kv heads")
@@ -379,7 +386,7 @@ def paged_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_tabl
                                    _ptr(block_tables), block_tables.shape[1], _ptr(row_q_start), _ptr(row_q_len),
                                    _ptr(row_ctx_len), rows, num_tokens, _ptr(out), tag(q), num_heads,
                                    num_kv_heads, head_dim, page_size, ctypes.c_float(scale),
-                                   int(window or 0), int(min_q_len), ctypes.c_longlong(k_cache.shape[0]),
+                                   int(window or 0), int(keep), int(min_q_len), ctypes.c_longlong(k_cache.shape[0]),
                                    int(out.dtype == torch.float32 and q.dtype != torch.float32), *(mods or _NO_MODS).args(num_heads),
                                    _stream()),
            "paged_attention")
@@ -389,7 +396,7 @@ def paged_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_tabl
 def prefill_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_tables, row_q_start, row_q_len,
                       row_ctx_len, num_tokens: int, out: torch.Tensor, num_heads: int, num_kv_heads: int,
                       head_dim: int, page_size: int, scale: float, window: int | None = None,
-                      min_q_len: int = 2, work=None, mods: ScoreMods | None = None) -> torch.Tensor:
+                      min_q_len: int = 2, work=None, mods: ScoreMods | None = None, keep: int = 0) -> torch.Tensor:
     """Causal attention of prompt portions over their request's pages (bfloat16, tensor cores).
     Rows with fewer than ``min_q_len`` new tokens are left alone.  ``work`` = (rows, tokens): how many rows have
     ``min_q_len`` tokens or more and their tokens in sum, where the caller knows -- the launch then has blocks for the
@@ -407,7 +414,7 @@ def prefill_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_ta
     _check(lib.mie_prefill_attention(_ptr(q), ctypes.c_int64(q_stride), _ptr(k_cache), _ptr(v_cache),
                                      _ptr(block_tables), block_tables.shape[1], _ptr(row_q_start), _ptr(row_q_len),
                                      _ptr(row_ctx_len), row_q_len.numel(), num_tokens, _ptr(out), num_heads,
-                                     num_kv_heads, head_dim, page_size, ctypes.c_float(scale), int(window or 0),
+                                     num_kv_heads, head_dim, page_size, ctypes.c_float(scale), int(window or 0), int(keep),
                                      int(min_q_len), ctypes.c_longlong(k_cache.shape[0]), *_work_args(work),
                                      int(out.dtype == torch.float32), *(mods or _NO_MODS).args(num_heads), _stream()),
            "prefill_attention")
@@ -417,7 +424,7 @@ def prefill_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_ta
 def prefill_attention_tc(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_tables, row_q_start, row_q_len,
                          row_ctx_len, num_tokens: int, out: torch.Tensor, num_heads: int, num_kv_heads: int,
                          head_dim: int, page_size: int, scale: float, window: int | None = None,
-                         min_q_len: int = 2, work=None, mods: ScoreMods | None = None) -> torch.Tensor:
+                         min_q_len: int = 2, work=None, mods: ScoreMods | None = None, keep: int = 0) -> torch.Tensor:
     """Causal attention of prompt portions on tcgen05 (S and O in tensor memory, operands by TMA);
     head_dim 64 or 128.  ``work``: as for ``prefill_attention``."""
     _need(q.dtype == torch.bfloat16 == k_cache.dtype == v_cache.dtype and out.dtype in (torch.bfloat16, torch.float32),
@@ -434,7 +441,7 @@ def prefill_attention_tc(q: torch.Tensor, q_stride: int, k_cache, v_cache, block
                                         ctypes.c_int64(k_cache.shape[0]), _ptr(block_tables), block_tables.shape[1],
                                         _ptr(row_q_start), _ptr(row_q_len), _ptr(row_ctx_len), row_q_len.numel(),
                                         num_tokens, _ptr(out), num_heads, num_kv_heads, head_dim, page_size,
-                                        ctypes.c_float(scale), int(window or 0), int(min_q_len), *_work_args(work),
+                                        ctypes.c_float(scale), int(window or 0), int(keep), int(min_q_len), *_work_args(work),
                                         int(out.dtype == torch.float32), *(mods or _NO_MODS).args(num_heads), _stream()),
            "prefill_attention_tc")
     return out
@@ -586,7 +593,7 @@ def decode_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_tab
                      row_ctx_len, out: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int,
                      page_size: int, scale: float, window: int | None = None, max_ctx: int = 0,
                      splits: int | None = None, merge: str | None = None, stages: int | None = None,
-                     tma: bool | None = None, min_part_tiles: int = 0, rope=None, mods: ScoreMods | None = None) -> torch.Tensor:
+                     tma: bool | None = None, min_part_tiles: int = 0, rope=None, mods: ScoreMods | None = None, keep: int = 0) -> torch.Tensor:
     """Attention of rows with exactly one new token (bfloat16, tensor cores, context split across
     blocks and merged in the same launch).  Rows with more new tokens are skipped.  ``merge`` =
     "cluster": 1, 2, 4 or 8 splits merged through distributed shared memory; "scratch": any number of
@@ -642,7 +649,7 @@ def decode_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_tab
     _check(lib.mie_decode_attention(_ptr(q), ctypes.c_int64(q_stride), _ptr(k_cache), _ptr(v_cache),
                                     _ptr(block_tables), block_tables.shape[1], _ptr(row_q_start), _ptr(row_q_len),
                                     _ptr(row_ctx_len), rows, _ptr(out), num_heads, num_kv_heads, head_dim,
-                                    page_size, ctypes.c_float(scale), int(window or 0), int(splits),
+                                    page_size, ctypes.c_float(scale), int(window or 0), int(keep), int(splits),
                                     _ptr(part_o), _ptr(part_lse), _ptr(counters), int(stages or 0),
                                     ctypes.c_int64(k_cache.shape[0] if tma else 0), ctypes.c_int64(k_cache.shape[0]),
                                     int(min_part_tiles if merge == "scratch" else 0),
@@ -756,12 +763,13 @@ def stream_norm(res: torch.Tensor, weight: torch.Tensor, groups: int, eps: float
 def qk_norm_rope(qkv: torch.Tensor, positions, slots, freq: torch.Tensor, q_out: torch.Tensor, k_cache, v_cache, *,
                  num_heads: int, num_kv_heads: int, dim: int, vdim: int, rot: int, page_size: int, eps: float = 0.0,
                  q_weight=None, k_weight=None, temp=None, q_scale: float = 1.0, k_scale: float = 1.0,
-                 write_cache: bool = True, head_norm: bool = False, interleaved: bool = False, pos_temp=None) -> torch.Tensor:
+                 write_cache: bool = True, head_norm: bool = False, interleaved: bool = False, pos_temp=None, v_freq=None) -> torch.Tensor:
     """From the fused projection rows [q: H x dim | k: G x dim | v: G x vdim | ...]: q and k optionally RMS-normed over
-    their whole projection (``head_norm``: per head, with ``dim`` weights shared by the heads), rotated by position x ``freq``
+    their whole projection (``head_norm``: per head, with ``dim`` weights shared by the heads or none), rotated by position x ``freq``
     over their first ``rot`` dims (pairs (i, i + rot/2), or (2i, 2i + 1) with ``interleaved``), q scaled per head and, with
     ``pos_temp`` = (coef, every), by 1 + coef ln(floor((position + 1) / every) + 1); q written to ``q_out`` [T, H, DP] and k, v
-    to their cache slots (pages [page, G, page_size, DP], tails zero)."""
+    to their cache slots (pages [page, G, page_size, DP], tails zero).  ``v_freq`` (vdim / 2): v is rotated too, over all its
+    dims, in the same pairing."""
     T = qkv.shape[0]
     DP = q_out.shape[-1]
     _need(qkv.dim() == 2 and qkv.stride(1) == 1
@@ -778,6 +786,9 @@ def qk_norm_rope(qkv: torch.Tensor, positions, slots, freq: torch.Tensor, q_out:
         _need(q_weight.numel() == (dim if head_norm else num_heads * dim), "q norm weight size")
     if k_weight is not None:
         _need(k_weight.numel() == (dim if head_norm else num_kv_heads * dim), "k norm weight size")
+    if v_freq is not None:
+        _need(vdim % 2 == 0, "values that rotate have an even size")
+        _f32(v_freq, "value frequencies", vdim // 2)
     coef, every = (float(pos_temp[0]), int(pos_temp[1])) if pos_temp else (0.0, 0)
     if temp is not None:
         _need(temp.numel() == num_heads, "one temperature per head")
@@ -786,8 +797,23 @@ def qk_norm_rope(qkv: torch.Tensor, positions, slots, freq: torch.Tensor, q_out:
                                 _ptr(q_weight), _ptr(k_weight), _ptr(temp), tag(ws[0]) if ws else 0, ctypes.c_float(eps),
                                 ctypes.c_float(q_scale), ctypes.c_float(k_scale), _ptr(q_out), _ptr(k_cache), _ptr(v_cache), T,
                                 num_heads, num_kv_heads, dim, vdim, DP, rot, page_size, ctypes.c_longlong(k_cache.shape[0]),
-                                int(write_cache), int(head_norm), int(interleaved), ctypes.c_float(coef), every, _stream()), "qk_norm_rope")
+                                int(write_cache), int(head_norm), int(interleaved), ctypes.c_float(coef), every, _ptr(v_freq), _stream()),
+           "qk_norm_rope")
     return q_out
+
+
+def turn_heads(attn: torch.Tensor, positions, freq: torch.Tensor, out: torch.Tensor, num_heads: int, vdim: int,
+               interleaved: bool = False) -> torch.Tensor:
+    """out[t, h * vdim + d]: heads of ``attn`` [T, H, DP >= vdim] with every pair of their ``vdim`` entries turned by -position x
+    ``freq`` (what undoes the rotation of values by their own positions, up to the difference of the two)."""
+    T, DP = attn.shape[0], attn.shape[-1]
+    _need(attn.is_contiguous() and attn.shape == (T, num_heads, DP) and DP >= vdim and vdim % 2 == 0, "attn must be [T, H, DP], the values of even size")
+    _need(out.is_contiguous() and out.shape == (T, num_heads * vdim) and out.dtype == attn.dtype, "out must be contiguous [T, H * vdim]")
+    _f32(freq, "value frequencies", vdim // 2)
+    _i32(positions, "positions")
+    _check(load("qk_norm_rope").mie_turn_heads(_ptr(attn), tag(attn), _ptr(positions), _ptr(freq), _ptr(out), T, num_heads, vdim, DP,
+                                               int(interleaved), _stream()), "turn_heads")
+    return out
 
 
 # --------------------------------------------------------------------------- retention
@@ -986,14 +1012,16 @@ def glu_clamped(gate_up: torch.Tensor, out: torch.Tensor, limit: float, slope: f
 
 def sigmoid_gate(attn: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, num_heads: int, vdim: int) -> torch.Tensor:
     """out[t, h * vdim + c] = attn[t, h, c] * sigmoid(gate[t, h * vdim + c]); ``attn`` [T, H, DP >= vdim], ``gate`` may be a
-    column slice of a wider tensor."""
+    column slice of a wider tensor.  A gate of H columns gates whole heads: sigmoid(gate[t, h])."""
     T, DP = attn.shape[0], attn.shape[-1]
     _need(attn.is_contiguous() and attn.shape == (T, num_heads, DP) and DP >= vdim, "attn must be [T, H, DP]")
-    _need(gate.stride(1) == 1 and gate.shape == (T, num_heads * vdim) and gate.dtype == attn.dtype == out.dtype, "gate must be [T, H * vdim]")
+    per_head = gate.shape[1] == num_heads and vdim > 1
+    _need(gate.stride(1) == 1 and gate.shape == (T, num_heads * (1 if per_head else vdim)) and gate.dtype == attn.dtype == out.dtype,
+          "gate must be [T, H * vdim] or [T, H]")
     _need(out.is_contiguous() and out.shape == (T, num_heads * vdim), "out must be contiguous [T, H * vdim]")
     lib = build.load("activation")
     _check(lib.mie_sigmoid_gate(_ptr(attn), _ptr(gate), ctypes.c_longlong(gate.stride(0)), _ptr(out), tag(out), T, num_heads, vdim, DP,
-                                _stream()), "sigmoid_gate")
+                                int(per_head), _stream()), "sigmoid_gate")
     return out
 
 
@@ -1041,31 +1069,35 @@ def hyper_norm(res: torch.Tensor, streams: int, out: torch.Tensor, *, weight=Non
 # --------------------------------------------------------------------------- latent attention
 
 def latent_norm_rope(down: torch.Tensor, positions, freq, q_weight, c_weight, eps: float, cq, c, kr, *, q_rank: int, kv_rank: int,
-                     rot_dim: int, rot: int) -> None:
+                     rot_dim: int, rot: int, interleaved: bool = True, gain: float = 1.0) -> None:
     """From rows [dq: q_rank | dkv: kv_rank + rot_dim | ...] of the down-projection: cq = rms(dq) q_weight, c =
     rms(dkv[:kv_rank]) c_weight (activation type), kr = dkv[kv_rank:] rotated by position x ``freq`` over its first ``rot``
-    entries, entry 2i with 2i + 1 (float32)."""
+    entries, entry 2i with 2i + 1 or (``interleaved`` False) i with i + rot / 2, cos and sin times ``gain`` (float32).  ``q_rank`` 0:
+    no query latent (``q_weight`` and ``cq`` None)."""
     T = down.shape[0]
     _need(down.dim() == 2 and down.stride(1) == 1 and down.shape[1] >= q_rank + kv_rank + rot_dim, "down-projection rows too short")
-    _f32(q_weight, "query latent norm weight", q_rank)
+    if q_rank:
+        _f32(q_weight, "query latent norm weight", q_rank)
+        _need(cq.shape == (T, q_rank) and cq.dtype == down.dtype and cq.is_contiguous(), "latents must be contiguous [T, rank] in the activation type")
     _f32(c_weight, "key/value latent norm weight", kv_rank)
     _f32(freq, "frequencies", rot // 2)
     _i32(positions, "positions")
-    _need(cq.shape == (T, q_rank) and c.shape == (T, kv_rank) and cq.dtype == c.dtype == down.dtype and cq.is_contiguous()
-          and c.is_contiguous(), "latents must be contiguous [T, rank] in the activation type")
+    _need(c.shape == (T, kv_rank) and c.dtype == down.dtype and c.is_contiguous(), "latents must be contiguous [T, rank] in the activation type")
     _need(kr.shape == (T, rot_dim) and kr.dtype == torch.float32 and kr.is_contiguous(), "the shared key part must be float32 [T, rot_dim]")
     lib = load("latent_kv")
     _check(lib.mie_latent_norm_rope(_ptr(down), tag(down), ctypes.c_longlong(down.stride(0)), _ptr(positions), _ptr(freq),
                                     _ptr(q_weight), _ptr(c_weight), ctypes.c_float(eps), _ptr(cq), _ptr(c), _ptr(kr), T, q_rank,
-                                    kv_rank, rot_dim, rot, _stream()), "latent_norm_rope")
+                                    kv_rank, rot_dim, rot, int(interleaved), ctypes.c_float(gain), _stream()), "latent_norm_rope")
 
 
 def latent_assemble(qu: torch.Tensor, kvu: torch.Tensor, kr: torch.Tensor, positions, slots, freq, q_out, k_cache, v_cache, *,
-                    num_heads: int, dim: int, rot_dim: int, vdim: int, rot: int, page_size: int, write_cache: bool = True) -> None:
+                    num_heads: int, dim: int, rot_dim: int, vdim: int, rot: int, page_size: int, write_cache: bool = True, interleaved: bool = True,
+                    gain: float = 1.0) -> None:
     """q_out[t, h] = [qu[t, h, :dim] | rotate(qu[t, h, dim:]) | 0]; cache k[h] = [kvu.k[h] | kr | 0], v[h] = [kvu.v[h] | 0]
-    with kvu rows [k: H x dim | v: H x vdim]; heads padded to the pages' width."""
+    with kvu rows [k: H x dim | v: H x vdim]; heads padded to the pages' width.  ``qu`` may be a column slice of a wider product;
+    ``interleaved``, ``gain``: as for ``latent_norm_rope``."""
     T, H, DP = qu.shape[0], num_heads, q_out.shape[-1]
-    _need(qu.is_contiguous() and qu.shape == (T, H * (dim + rot_dim)), "qu must be contiguous [T, H * (dim + rot_dim)]")
+    _need(qu.stride(1) == 1 and qu.shape == (T, H * (dim + rot_dim)), "qu must be rows of H * (dim + rot_dim)")
     _need(kvu.is_contiguous() and kvu.shape == (T, H * (dim + vdim)) and kvu.dtype == qu.dtype, "kvu must be contiguous [T, H * (dim + vdim)]")
     _need(kr.shape == (T, rot_dim) and kr.dtype == torch.float32 and kr.is_contiguous(), "the shared key part must be float32 [T, rot_dim]")
     _need(q_out.is_contiguous() and q_out.shape == (T, H, DP) and q_out.dtype == qu.dtype, "q_out must be [T, H, DP]")
@@ -1075,9 +1107,10 @@ def latent_assemble(qu: torch.Tensor, kvu: torch.Tensor, kr: torch.Tensor, posit
     _i32(positions, "positions")
     _i32(slots, "slots")
     lib = load("latent_kv")
-    _check(lib.mie_latent_assemble(_ptr(qu), _ptr(kvu), tag(qu), _ptr(kr), _ptr(positions), _ptr(slots), _ptr(freq), _ptr(q_out),
+    _check(lib.mie_latent_assemble(_ptr(qu), ctypes.c_longlong(qu.stride(0)), _ptr(kvu), tag(qu), _ptr(kr), _ptr(positions), _ptr(slots), _ptr(freq), _ptr(q_out),
                                    _ptr(k_cache), _ptr(v_cache), T, H, dim, rot_dim, vdim, DP, rot, page_size,
-                                   ctypes.c_longlong(k_cache.shape[0]), int(write_cache), _stream()), "latent_assemble")
+                                   ctypes.c_longlong(k_cache.shape[0]), int(write_cache), int(interleaved), ctypes.c_float(gain),
+                                   _stream()), "latent_assemble")
 
 
 # --------------------------------------------------------------------------- differential attention

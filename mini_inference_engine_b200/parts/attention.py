@@ -97,17 +97,23 @@ class GatedAttention(Mixer):
     * ``qk_norm``: q and k are RMS-normed over their whole projection (all heads at once) with weights 'q.norm', 'k.norm';
     * rotation over the first ``rot_dims`` dims with frequencies that may be rescaled by wavelength (``rot_scaling``);
     * ``head_temp``: the score of head h is multiplied by 'temp'[h] (folded into the query);
-    * ``chunk``: a query sees keys of its own block of that many positions only; ``window``: a sliding window;
+    * ``chunk``: a query sees keys of its own block of that many positions only; ``window``: a sliding window; ``keep_first``: with
+      either, the first that many keys of the sequence stay in sight (their pages are never given back);
     * ``gate``: the concatenated heads are multiplied by sigmoid(W_g h) before the output projection;
     * ``bias``: q, k and v have biases 'q.b', 'k.b', 'v.b', added in the projection;
-    * ``qk_norm`` "head": the RMS norm is per head, with ``dim`` weights ('q.norm', 'k.norm') shared by all heads;
+    * ``qk_norm`` "head": the RMS norm is per head, with ``dim`` weights ('q.norm', 'k.norm') shared by all heads; "unit": per head and
+      without weights (whether before or after the rotation is the same: it leaves a head's root mean square as it is);
+    * ``rot_scaling``: frequencies rescaled (parts.rope.rotary_frequencies: by wavelength, linearly);
+    * ``rotate_values``: the value at position j is rotated by j over all its dims (unscaled frequencies of ``rot_base``, the same
+      pairing) before it is stored, and a head's output at position i is turned back by i: values mix by relative position;
     * ``rot_pairing`` "interleaved": the rotation pairs entry 2i with 2i + 1 (default: i with i + rot_dims / 2);
     * ``q_temp`` (coef, every): the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1);
     * ``softcap`` c: score <- c tanh(score / c) after the scale;
     * ``rel_bias`` (rows, far): a learned bias 'rel' [rows, heads] by distance n = p - j is added to the (scaled, capped) score:
       row n for n < rows / 2, else min(rows - 1, rows/2 + floor(ln(n / (rows/2)) / ln(far / (rows/2)) (rows - rows/2)));
       ``rows`` None: the table's rows come from the checkpoint's tensor (a random model gets 32);
-    * ``sink``: a learned number per head ('sink') whose exponential is one more term of the softmax's denominator (nothing is scored for it, nothing read).
+    * ``sink``: a learned number per head ('sink') whose exponential is one more term of the softmax's denominator (nothing is scored for it,
+      nothing read); "one": the term is 1 (a score of 0) for every head and nothing is learned.
 
     q, k, v and the gate are one product; norm, rotation, temperature and the cache write one kernel; attention
     itself is the framework's paged kernels (decode and portions); the gate one more."""
@@ -116,14 +122,23 @@ class GatedAttention(Mixer):
                  rot_dims: int, rot_base: float, eps: float, rot_scaling: dict | None = None, qk_norm: bool = True,
                  head_temp: bool = True, gate: bool = True, chunk: int | None = None, window: int | None = None,
                  bias: bool = False, rot_pairing: str = "half", q_temp=None, softcap: float = 0.0, rel_bias=None,
-                 sink: bool = False):
+                 sink=False, rotate_values: bool = False, keep_first: int = 0):
         if rot_pairing not in ("half", "interleaved"):
             raise ValueError(f"rot_pairing {rot_pairing!r}; half or interleaved")
-        if qk_norm not in (True, False, "head", "projection"):
-            raise ValueError(f"qk_norm {qk_norm!r}; False, True / 'projection' or 'head'")
+        if qk_norm not in (True, False, "head", "projection", "unit"):
+            raise ValueError(f"qk_norm {qk_norm!r}; False, True / 'projection', 'head' or 'unit'")
+        if sink not in (True, False, "one"):
+            raise ValueError(f"sink {sink!r}; False, True or 'one'")
+        if rot_scaling is not None and rot_scaling.get("kind") == "yarn":
+            raise ValueError("this attention's rotation keeps lengths; yarn scales cos and sin (LatentAttention takes it)")
+        if rotate_values and vdim % 2:
+            raise ValueError(f"values of {vdim} entries do not rotate in pairs")
+        if keep_first < 0:
+            raise ValueError("keep_first must not be negative")
         if rel_bias is not None and rel_bias[0] is not None and (int(rel_bias[0]) < 2 or float(rel_bias[1]) <= int(rel_bias[0]) // 2):
             raise ValueError(f"rel_bias {rel_bias!r}: two rows or more, and a far distance beyond half of them")
-        self.bias, self.rot_pairing, self.softcap, self.sink = bool(bias), rot_pairing, float(softcap or 0.0), bool(sink)
+        self.bias, self.rot_pairing, self.softcap, self.sink = bool(bias), rot_pairing, float(softcap or 0.0), sink
+        self.rotate_values, self.keep_first = bool(rotate_values), int(keep_first) if window or chunk else 0
         self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp else None
         self.rel_bias = (int(rel_bias[0]) if rel_bias[0] is not None else None, float(rel_bias[1])) if rel_bias else None
         if num_heads % num_kv_heads:
@@ -137,7 +152,7 @@ class GatedAttention(Mixer):
         self.scale, self.eps = float(scale), eps
         self.rot_dims, self.rot_base, self.rot_scaling = rot_dims, rot_base, rot_scaling
         self.qk_norm, self.head_temp, self.gate, self.chunk, self.window = qk_norm, head_temp, gate, chunk, window
-        self.need = KVNeed(num_kv_heads, self.padded, window, chunk)
+        self.need = KVNeed(num_kv_heads, self.padded, window, chunk, self.keep_first)
 
     def tensor_specs(self):
         H, G, D, Dv, h = self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.hidden_size
@@ -147,7 +162,7 @@ class GatedAttention(Mixer):
             specs["g"] = TensorSpec((H * Dv, h), "fan_in")
         if self.qk_norm == "head":
             specs.update({"q.norm": TensorSpec((D,), "normal:1:0.1"), "k.norm": TensorSpec((D,), "normal:1:0.1")})
-        elif self.qk_norm:
+        elif self.qk_norm in (True, "projection"):
             specs.update({"q.norm": TensorSpec((H * D,), "normal:1:0.1"), "k.norm": TensorSpec((G * D,), "normal:1:0.1")})
         if self.head_temp:
             specs["temp"] = TensorSpec((H,), "uniform:0.5:2")
@@ -156,7 +171,7 @@ class GatedAttention(Mixer):
                           "v.b": TensorSpec((G * Dv,), "normal:0:0.1")})
         if self.rel_bias:
             specs["rel"] = TensorSpec((self.rel_bias[0] or -1, H), "normal:0:1", (self.rel_bias[0] or 32, H))
-        if self.sink:
+        if self.sink is True:
             specs["sink"] = TensorSpec((H,), "normal:0:1")
         return specs
 
@@ -169,10 +184,12 @@ class GatedAttention(Mixer):
         self.w_in = rt.place(torch.cat(parts, 0))
         self.w_o = rt.place(tensors["o"])
         small = lambda n: tensors[n].float().to(rt.device).contiguous()        # read as float32 by the kernel
-        self.q_norm = small("q.norm") if self.qk_norm else None
-        self.k_norm = small("k.norm") if self.qk_norm else None
+        weighted = self.qk_norm and self.qk_norm != "unit"
+        self.q_norm = small("q.norm") if weighted else None
+        self.k_norm = small("k.norm") if weighted else None
         self.temp = small("temp") if self.head_temp else None
         self.freq = rotary_frequencies(self.rot_dims, self.rot_base, self.rot_scaling).to(rt.device)
+        self.v_freq = rotary_frequencies(self.vdim, self.rot_base).to(rt.device) if self.rotate_values else None
         self.b_in = None
         if self.bias:
             b = torch.cat([tensors[n].float() for n in ("q.b", "k.b", "v.b")])
@@ -193,7 +210,10 @@ class GatedAttention(Mixer):
         from ..kernels import ops
         self.mods = None
         if self.softcap > 0 or self.sink or dist is not None:
-            self.mods = ops.ScoreMods(self.softcap, small("sink") if self.sink else None, dist)
+            term = None
+            if self.sink:
+                term = small("sink") if self.sink is True else torch.zeros(self.num_heads, dtype=torch.float32, device=rt.device)
+            self.mods = ops.ScoreMods(self.softcap, term, dist)
 
     def cache_need(self):
         return self.need
@@ -215,9 +235,14 @@ class GatedAttention(Mixer):
         ops.qk_norm_rope(proj, ctx.positions, ctx.slots[cache.group], self.freq, q, cache.k, cache.v, num_heads=H,
                          num_kv_heads=G, dim=D, vdim=Dv, rot=self.rot_dims, page_size=cache.page_size, eps=self.eps,
                          q_weight=self.q_norm, k_weight=self.k_norm, temp=self.temp, write_cache=cache.writes,
-                         head_norm=self.qk_norm == "head", interleaved=self.rot_pairing == "interleaved", pos_temp=self.q_temp)
+                         head_norm=self.qk_norm in ("head", "unit"), v_freq=self.v_freq, interleaved=self.rot_pairing == "interleaved", pos_temp=self.q_temp)
         heads = self.rt.empty(T, H, DP)
-        attn_kernels.attention(q, ctx, cache, heads, H, G, DP, self.scale, self.need.mask(), q_stride=H * DP, mods=self.mods)
+        attn_kernels.attention(q, ctx, cache, heads, H, G, DP, self.scale, self.need.mask(), q_stride=H * DP, mods=self.mods,
+                               keep=self.keep_first)
+        if self.rotate_values:
+            turned = self.rt.empty(T, H * Dv)
+            ops.turn_heads(heads, ctx.positions, self.v_freq, turned, H, Dv, interleaved=self.rot_pairing == "interleaved")
+            heads, DP = turned.view(T, H, Dv), Dv
         if self.gate or DP != Dv:
             gated = self.rt.empty(T, H * Dv)
             if self.gate:
@@ -336,13 +361,23 @@ class LatentAttention(Mixer):
     pairs entry 2i with 2i + 1 over the first ``rot_dims`` entries of the rotated part.  Causal softmax attention, an
     output gate sigmoid(W_g h) on the concatenated heads, then W_o.
 
-    The down-projections and the gate are one product; both RMS norms and the rotation of the shared key part one
+    ``q_rank`` None: no query latent, q = W_q h ('q').  ``rot_pairing`` "half": the rotation pairs i with i + rot_dims / 2.
+    ``rot_scaling``: rescaled frequencies (parts.rope.rotary_frequencies; "yarn" also scales cos and sin).  ``sink``: a learned
+    number per head whose exponential joins the softmax's denominator.  ``gate`` "head": one gate logit a head, 'g' [H, hidden].
+
+    The down-projections (or q and the down-projection) and the gate are one product; both RMS norms and the rotation of the shared key part one
     kernel; the up-projections of keys and values one product; queries and keys are put together per head (and keys
     and values written to the pages) by one more kernel, after which the framework's paged attention kernels run with as
     many key/value heads as query heads."""
 
-    def __init__(self, hidden_size: int, num_heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int,
-                 scale: float, rot_dims: int, rot_base: float, eps: float, gate: bool = True, window: int | None = None):
+    def __init__(self, hidden_size: int, num_heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int | None, kv_rank: int,
+                 scale: float, rot_dims: int, rot_base: float, eps: float, gate=True, window: int | None = None,
+                 rot_pairing: str = "interleaved", rot_scaling: dict | None = None, sink: bool = False):
+        if rot_pairing not in ("half", "interleaved"):
+            raise ValueError(f"rot_pairing {rot_pairing!r}; half or interleaved")
+        if gate not in (True, False, "head"):
+            raise ValueError(f"gate {gate!r}; True, False or 'head'")
+        self.rot_pairing, self.rot_scaling, self.sink = rot_pairing, rot_scaling, bool(sink)
         if rot_dims % 2 or rot_dims > rot_dim:
             raise ValueError(f"rot_dims {rot_dims} must be even and at most rot_dim {rot_dim}")
         self.hidden_size, self.num_heads, self.dim, self.rot_dim, self.vdim = hidden_size, num_heads, dim, rot_dim, vdim
@@ -355,57 +390,69 @@ class LatentAttention(Mixer):
 
     def tensor_specs(self):
         H, D, R, Dv, h = self.num_heads, self.dim, self.rot_dim, self.vdim, self.hidden_size
-        specs = {"dq": TensorSpec((self.q_rank, h), "fan_in"), "dq.norm": TensorSpec((self.q_rank,), "normal:1:0.1"),
-                 "uq": TensorSpec((H * (D + R), self.q_rank), "fan_in"), "dkv": TensorSpec((self.kv_rank + R, h), "fan_in"),
+        if self.q_rank:
+            specs = {"dq": TensorSpec((self.q_rank, h), "fan_in"), "dq.norm": TensorSpec((self.q_rank,), "normal:1:0.1"),
+                     "uq": TensorSpec((H * (D + R), self.q_rank), "fan_in")}
+        else:
+            specs = {"q": TensorSpec((H * (D + R), h), "fan_in")}
+        specs.update({"dkv": TensorSpec((self.kv_rank + R, h), "fan_in"),
                  "dkv.norm": TensorSpec((self.kv_rank,), "normal:1:0.1"), "uk": TensorSpec((H * D, self.kv_rank), "fan_in"),
-                 "uv": TensorSpec((H * Dv, self.kv_rank), "fan_in"), "o": TensorSpec((h, H * Dv), "fan_in")}
+                 "uv": TensorSpec((H * Dv, self.kv_rank), "fan_in"), "o": TensorSpec((h, H * Dv), "fan_in")})
         if self.gate:
-            specs["g"] = TensorSpec((H * Dv, h), "fan_in")
+            specs["g"] = TensorSpec((H if self.gate == "head" else H * Dv, h), "fan_in")
+        if self.sink:
+            specs["sink"] = TensorSpec((H,), "normal:0:1")
         return specs
 
     def bind(self, tensors, rt):
-        from .rope import rotary_frequencies
+        from ..kernels import ops
+        from .rope import rotary_frequencies, rotary_gain
         self.rt = rt
-        w, _ = _padded_rows([tensors["dq"], tensors["dkv"]] + ([tensors["g"]] if self.gate else []))
+        w, _ = _padded_rows([tensors["dq" if self.q_rank else "q"], tensors["dkv"]] + ([tensors["g"]] if self.gate else []))
         self.w_down = rt.place(w)
-        self.w_uq = rt.place(tensors["uq"])
+        self.w_uq = rt.place(tensors["uq"]) if self.q_rank else None
         uk, uv = tensors["uk"], tensors["uv"]
         if uk.dtype != uv.dtype:
             uk, uv = uk.float(), uv.float()
         self.w_ukv = rt.place(torch.cat([uk, uv], 0))
         self.w_o = rt.place(tensors["o"])
         small = lambda n: tensors[n].float().to(rt.device).contiguous()
-        self.q_norm, self.c_norm = small("dq.norm"), small("dkv.norm")
-        self.freq = rotary_frequencies(self.rot_dims, self.rot_base).to(rt.device)
+        self.q_norm, self.c_norm = small("dq.norm") if self.q_rank else None, small("dkv.norm")
+        self.freq = rotary_frequencies(self.rot_dims, self.rot_base, self.rot_scaling).to(rt.device)
+        self.gain = rotary_gain(self.rot_scaling)
+        self.mods = ops.ScoreMods(sink=small("sink")) if self.sink else None
 
     def cache_need(self):
         return self.need
 
     def kernel_sources(self):
-        return (self.rt.product_sources(self.w_down, self.w_uq, self.w_ukv, self.w_o) | {"latent_kv", "activation"}
+        return (self.rt.product_sources(*(w for w in (self.w_down, self.w_uq, self.w_ukv, self.w_o) if w is not None)) | {"latent_kv", "activation"}
                 | _attention_sources(self.rt, self.padded))
 
     def forward(self, x, ctx, cache):
         from ..kernels import ops
         H, D, R, Dv, DP = self.num_heads, self.dim, self.rot_dim, self.vdim, self.padded
         T = ctx.num_tokens
+        interleaved, q_rank = self.rot_pairing == "interleaved", self.q_rank or 0
+        q_cols = q_rank or H * (D + R)                            # the columns in front of the key/value latent's
         down = self.rt.linear(x, self.w_down)
-        cq, c = self.rt.empty(T, self.q_rank), self.rt.empty(T, self.kv_rank)
+        cq, c = self.rt.empty(T, q_rank) if q_rank else None, self.rt.empty(T, self.kv_rank)
         kr = self.rt.empty(T, R, dtype=torch.float32)
-        ops.latent_norm_rope(down, ctx.positions, self.freq, self.q_norm, self.c_norm, self.eps, cq, c, kr, q_rank=self.q_rank,
-                             kv_rank=self.kv_rank, rot_dim=R, rot=self.rot_dims)
-        qu = self.rt.linear(cq, self.w_uq)
+        ops.latent_norm_rope(down if q_rank else down[:, q_cols:], ctx.positions, self.freq, self.q_norm, self.c_norm, self.eps, cq, c, kr,
+                             q_rank=q_rank, kv_rank=self.kv_rank, rot_dim=R, rot=self.rot_dims, interleaved=interleaved, gain=self.gain)
+        qu = self.rt.linear(cq, self.w_uq) if q_rank else down[:, :q_cols]
         kvu = self.rt.linear(c, self.w_ukv)
         q = self.rt.empty(T, H, DP)
         ops.latent_assemble(qu, kvu, kr, ctx.positions, ctx.slots[cache.group], self.freq, q, cache.k, cache.v, num_heads=H, dim=D,
-                            rot_dim=R, vdim=Dv, rot=self.rot_dims, page_size=cache.page_size, write_cache=cache.writes)
+                            rot_dim=R, vdim=Dv, rot=self.rot_dims, page_size=cache.page_size, write_cache=cache.writes,
+                            interleaved=interleaved, gain=self.gain)
         heads = self.rt.empty(T, H, DP)
-        attn_kernels.attention(q, ctx, cache, heads, H, H, DP, self.scale, self.need.mask(), q_stride=H * DP)
+        attn_kernels.attention(q, ctx, cache, heads, H, H, DP, self.scale, self.need.mask(), q_stride=H * DP, mods=self.mods)
         if self.gate or DP != Dv:
             gated = self.rt.empty(T, H * Dv)
             if self.gate:
-                at = self.q_rank + self.kv_rank + R
-                ops.sigmoid_gate(heads, down[:, at:at + H * Dv], gated, H, Dv)
+                at = q_cols + self.kv_rank + R
+                ops.sigmoid_gate(heads, down[:, at:at + (H if self.gate == "head" else H * Dv)], gated, H, Dv)
             else:
                 gated.view(T, H, Dv).copy_(heads[:, :, :Dv])
         else:

@@ -68,6 +68,25 @@ class PreNormResidual(Block):
 register_part("block", "prenorm_residual", PreNormResidual)
 
 
+class ParallelResidual(Block):
+    """One norm, both sublayers on its output, one sum: h = norm(x), x <- x + mixer(h) + ff(h).  The two sublayers depend on nothing
+    of one another and run side by side (two streams between a fork and a join; two arms of a captured step); the sum of the
+    stream and both outputs is fused into the next norm.  ``feed_forward`` may be absent."""
+    roles = {"mixer": "mixer", "feed_forward": "feed_forward", "norm": "norm"}
+    optional_roles = ("feed_forward",)
+
+    def forward(self, delta, res, ctx, cache):
+        from .parallel import side_by_side
+        x = self.norm(delta, res)
+        ff = getattr(self, "feed_forward", None)
+        if ff is None:
+            return self.mixer.forward(x, ctx, cache)
+        return Branches(side_by_side(x, lambda: self.mixer.forward(x, ctx, cache), lambda: ff.forward(x, ctx)))
+
+
+register_part("block", "parallel_residual", ParallelResidual)
+
+
 class Branches:
     """What a mixer may return instead of one tensor: several outputs that the block's norm adds together, each
     optionally RMS-normed over its row with ``inner_weights[k]`` first, the sum multiplied by ``coef``."""

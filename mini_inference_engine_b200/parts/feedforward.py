@@ -106,22 +106,27 @@ register_part("feed_forward", "clamped_glu", ClampedGLU)
 
 
 class ActivatedMLP(FeedForward):
-    """A feed-forward without a gate: W_down act(W_up h).  ``activation`` "xielu": two learned numbers p, q in the tensor
+    """A feed-forward without a gate: W_down act(W_up h).  ``activation`` "relu2": the square of relu.  "xielu": two learned numbers p, q in the tensor
     'act' [2]; for z > 0, softplus(p) z^2 + z / 2; for z <= 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2.  The last
     product leaves float32 for the stream's sum."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "xielu"):
-        if activation != "xielu":
-            raise ValueError(f"activation {activation!r}; this feed-forward has xielu")
+        if activation not in ("xielu", "relu2"):
+            raise ValueError(f"activation {activation!r}; this feed-forward has xielu and relu2")
         self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
 
     def tensor_specs(self):
         h, i = self.hidden_size, self.intermediate_size
-        return {"up": TensorSpec((i, h), "fan_in"), "down": TensorSpec((h, i), "fan_in"), "act": TensorSpec((2,), "normal:0:0.5")}
+        specs = {"up": TensorSpec((i, h), "fan_in"), "down": TensorSpec((h, i), "fan_in")}
+        if self.activation == "xielu":
+            specs["act"] = TensorSpec((2,), "normal:0:0.5")
+        return specs
 
     def bind(self, tensors, rt):
         self.rt = rt
         self.w_up, self.w_down = rt.place(tensors["up"]), rt.place(tensors["down"])
+        if self.activation != "xielu":
+            return
         p, q = tensors["act"].double().tolist()              # constants of the model: their softplus once, in 64-bit
         softplus = lambda z: max(z, 0.0) + math.log1p(math.exp(-abs(z)))
         self.ap, self.an = softplus(p), 0.5 + softplus(q)
@@ -130,7 +135,11 @@ class ActivatedMLP(FeedForward):
         return {"activation"} | self.rt.product_sources(self.w_up, self.w_down)
 
     def forward(self, x, ctx):
-        act = linear_kernels.linear_xielu(x, self.w_up, self.ap, self.an, self.rt.dtype)      # the activation in the product's epilogue
+        # the activation in the product's epilogue
+        if self.activation == "relu2":
+            act = linear_kernels.linear_relu2(x, self.w_up, self.rt.dtype)
+        else:
+            act = linear_kernels.linear_xielu(x, self.w_up, self.ap, self.an, self.rt.dtype)
         return self.rt.linear(act, self.w_down, None, out_dtype=torch.float32)
 
 

@@ -24,6 +24,26 @@ def _side_stream(device):
     return _side_streams[key]
 
 
+def side_by_side(x, first, second) -> list:
+    """[first(), second()], two pieces of work that depend on nothing of one another, the second on a stream of its own between
+    a fork and a join (events; inside a captured step they become two arms of the graph).  A decode step is a chain of
+    short kernels, and two chains side by side take the time of the longer one.  Every tensor either arm
+    makes is used by the main stream only after the join, and the side stream starts only after the fork,
+    so the allocator's per-stream reuse stays ordered.  The arms must not share a kernel's scratch memory."""
+    if not (SIDE_BY_SIDE_STREAMS and x.is_cuda):
+        return [first(), second()]
+    main, side = torch.cuda.current_stream(), _side_stream(x.device)
+    fork, join = torch.cuda.Event(), torch.cuda.Event()
+    fork.record(main)
+    side.wait_event(fork)
+    with torch.cuda.stream(side):
+        b = second()
+        join.record(side)
+    a = first()
+    main.wait_event(join)
+    return [a, b]
+
+
 class ParallelMixers(Mixer):
     def __init__(self, hidden_size: int, branches: dict, scales=None):
         """``branches``: {name: PartSpec of a mixer}; a branch's tensors are '<name>.<its own>', its out-norm weight
@@ -65,23 +85,9 @@ class ParallelMixers(Mixer):
         return names
 
     def forward(self, x, ctx, cache):
-        if (len(self.branches) == 2 and SIDE_BY_SIDE_STREAMS and x.is_cuda
-                and type(self.branches[0]) is not type(self.branches[1])):      # two of a kind would share their kernels' scratch
-            # The branches depend on nothing of one another: the second runs on a stream of its own between a fork and a
-            # join (events; inside a captured step they become two arms of the graph).  A decode step is a chain of
-            # short kernels, and two chains of five side by side take the time of one.  Every tensor either branch
-            # makes is used by the main stream only after the join, and the side stream starts only after the fork,
-            # so the allocator's per-stream reuse stays ordered.
-            main, side = torch.cuda.current_stream(), _side_stream(x.device)
-            fork, join = torch.cuda.Event(), torch.cuda.Event()
-            fork.record(main)
-            side.wait_event(fork)
-            with torch.cuda.stream(side):
-                second = self.branches[1].forward(x, ctx, cache.parts[1])
-                join.record(side)
-            first = self.branches[0].forward(x, ctx, cache.parts[0])
-            main.wait_event(join)
-            outs = [first, second]
+        if len(self.branches) == 2 and type(self.branches[0]) is not type(self.branches[1]):      # two of a kind would share their kernels' scratch
+            outs = side_by_side(x, lambda: self.branches[0].forward(x, ctx, cache.parts[0]),
+                                lambda: self.branches[1].forward(x, ctx, cache.parts[1]))
         else:
             outs = [b.forward(x, ctx, c) for b, c in zip(self.branches, cache.parts)]
         if self.scales is not None:

@@ -11,6 +11,7 @@ keys and values into their cache slots, which the reference does right after it
 """
 from __future__ import annotations
 
+import math
 import os
 
 import torch
@@ -93,15 +94,32 @@ register_part("position", "none", NoPosition)
 
 def rotary_frequencies(dims: int, base: float, scaling: dict | None = None) -> torch.Tensor:
     """float32 frequencies f_i = base^(-2i/dims), i < dims/2, for kernels that compute angles from positions
-    themselves (no table, no bound on the position).  ``scaling`` = {factor, low, high, original} rescales by
-    wavelength l = 2 pi / f: waves shorter than original/high keep their frequency, waves longer than
-    original/low get f / factor, and between the two the frequency is the blend (1 - s) f / factor + s f with
-    s = (original / l - low) / (high - low)."""
-    import math
+    themselves (no table, no bound on the position).  ``scaling`` may rescale them; its ``kind`` says how:
+
+    * "wavelength" (the default), {factor, low, high, original}: by wavelength l = 2 pi / f, waves shorter than original/high
+      keep their frequency, waves longer than original/low get f / factor, and between the two the frequency is the blend
+      (1 - s) f / factor + s f with s = (original / l - low) / (high - low);
+    * "linear", {factor}: every f_i / factor;
+    * "yarn", {factor, original, fast, slow}: the pair that makes t turns over ``original`` positions has the index
+      d(t) = dims ln(original / (2 pi t)) / (2 ln base); pairs up to floor(d(fast)) keep their frequency, pairs from ceil(d(slow))
+      on get f / factor, and between the two the share of f / factor grows linearly with the index.  (cos and sin of such a
+      rotation are also scaled: ``rotary_gain``.)"""
+    kind = (scaling or {}).get("kind", "wavelength")
+    if kind not in ("wavelength", "linear", "yarn"):
+        raise ValueError(f"rotary scaling {kind!r}; wavelength, linear or yarn")
+    if scaling and kind == "yarn":
+        factor, orig, fast, slow = (float(scaling[k]) for k in ("factor", "original", "fast", "slow"))
+        index = lambda turns: dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(float(base)))
+        lo, hi = max(math.floor(index(fast)), 0), min(math.ceil(index(slow)), dims - 1)
     out = []
     for i in range(dims // 2):
         f = float(base) ** (-2.0 * i / dims)
-        if scaling:
+        if scaling and kind == "linear":
+            f = f / float(scaling["factor"])
+        elif scaling and kind == "yarn":
+            share = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            f = f / factor * share + f * (1.0 - share)
+        elif scaling:
             factor, low, high, orig = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
             wave = 2.0 * math.pi / f
             if wave > orig / low:
@@ -111,3 +129,8 @@ def rotary_frequencies(dims: int, base: float, scaling: dict | None = None) -> t
                 f = (1.0 - s) * f / factor + s * f
         out.append(f)
     return torch.tensor(out, dtype=torch.float32)
+
+
+def rotary_gain(scaling: dict | None) -> float:
+    """What cos and sin of a rescaled rotation are multiplied by: 0.1 ln(factor) + 1 for "yarn", 1 for the others."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling and scaling.get("kind") == "yarn" else 1.0
