@@ -473,12 +473,29 @@ def luluzen_configs(size: dict, vocab=32000, positions=4096):
     return luluzen, design_configs(size, vocab, positions)[1]
 
 
+def radenex_configs(size: dict, vocab=32000, positions=4096):
+    """A Radenex configuration of the given layer sizes -- windowed attention that keeps the first tokens (rotated values, heads of
+    unit root mean square) and two layers of latent attention (96 plain and 32 rotated dims a head, values of 128) as a
+    stretch that runs twice: six layer runs, every one with a squared-relu feed-forward whose two matrices are as large as
+    Llama's three -- and the Llama configuration with the same width, heads and number of layers."""
+    from mini_inference_engine_b200.config import load_config
+    w, ff, H, G = size["width"], size["ff"], size["heads"], size["kv_heads"]
+    mlp = dict(kind="dense", ff=(3 * ff // 2 + 63) // 64 * 64)
+    win = dict(type="attention", mlp=mlp, mixer=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024, keep_first=64),
+                                                     rot=dict(base=5e5, dims=64, scaling=dict(factor=2.0))))
+    lat = dict(type="latent_attention", mlp=mlp, mixer=dict(heads=H, dim=96, rot_dim=32, vdim=128, kv_rank=w // 4, scale=128 ** -0.5,
+                                                            rot=dict(base=5e5, dims=32, scaling=dict(factor=8.0, original=positions, fast=32.0, slow=1.0))))
+    radenex = load_config(dict(architecture="Radenex", vocab=vocab, width=w, norm=dict(eps=1e-5), loop=dict(start=0, stop=3, times=2),
+                               layers=[win, lat, lat]))
+    return radenex, design_configs(size, vocab, positions)[1]
+
+
 KERNEL_FACES = ("embedding", "add_rmsnorm", "stream_norm", "rope_cache_write", "qk_norm_rope", "paged_attention", "prefill_attention",
                 "prefill_attention_tc", "decode_attention", "retention_scan", "head_rms_gate", "causal_conv", "recurrence_gates",
                 "recurrence_scan", "swiglu", "glu_clamped", "sigmoid_gate", "hyper_norm", "latent_norm_rope", "latent_assemble",
                 "diff_combine", "delta_prepare", "conv_state_update", "delta_scan", "head_norm_gate", "moe_route", "moe_router", "moe_dense_act", "moe_pairs", "moe_sort", "moe_gather", "moe_act_rows", "moe_combine", "grouped_linear",
                 "pair_embedding", "normed_add", "xielu", "gelu_gate_rows", "moe_glu", "add_layernorm", "stream_join", "tanh_cap",
-                "decay_scan", "gate_scan", "group_norm_gate")
+                "decay_scan", "gate_scan", "group_norm_gate", "turn_heads", "relu2")
 
 
 class KernelTimes:
@@ -503,7 +520,7 @@ class KernelTimes:
 
     def __enter__(self):
         from mini_inference_engine_b200.kernels import linear, ops
-        for mod, names in ((ops, KERNEL_FACES), (linear, ("linear", "linear_swiglu", "linear_into_stream"))):
+        for mod, names in ((ops, KERNEL_FACES), (linear, ("linear", "linear_swiglu", "linear_relu2", "linear_into_stream"))):
             for n in names:
                 self._saved.append((mod, n, getattr(mod, n)))
                 setattr(mod, n, self._wrap(n, getattr(mod, n)))
@@ -533,7 +550,8 @@ def run_design(args, steps, warmup):
     from mini_inference_engine_b200 import EngineConfig, LLMEngine
     from mini_inference_engine_b200.weights import write_model_folder
     pk = peaks()
-    configs_for = {"getizen": design_configs, "kebudra": kebudra_configs, "serotar": serotar_configs, "luluzen": luluzen_configs}[args.design]
+    configs_for = {"getizen": design_configs, "kebudra": kebudra_configs, "serotar": serotar_configs, "luluzen": luluzen_configs,
+                   "radenex": radenex_configs}[args.design]
     out = {"metric": "design_comparison", "design": args.design.capitalize(), "beside": "Llama", "dtype": "bf16", "data": "synthetic (random weights, seed 0)",
            "peaks": pk, "sizes": {}}
     batches = [int(b) for b in args.points.split(",") if b] or [8]
@@ -599,7 +617,7 @@ def main():
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the configuration has (named in config)")
     ap.add_argument("--preset", default="tinyllama-1.1b")
     ap.add_argument("--points", default="1,64", help="further decode batch sizes, comma separated ('' for none)")
-    ap.add_argument("--design", default=None, choices=["getizen", "kebudra", "serotar", "luluzen"],
+    ap.add_argument("--design", default=None, choices=["getizen", "kebudra", "serotar", "luluzen", "radenex"],
                     help="instead of the default workload: prefill and decode throughput of this design beside Llama at equal "
                          "layer sizes (--sizes), random weights; decode batches from --points")
     ap.add_argument("--sizes", default="w2048,w4096", help="with --design: layer sizes to measure, of " + ", ".join(DESIGN_SIZES))
