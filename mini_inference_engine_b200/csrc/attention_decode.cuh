@@ -1,6 +1,7 @@
-// The decode attention kernel, its parameter block and its launch by head size, shared by the two
-// entry points that differ only in where the scratch memory comes from (attention_decode.cu: the
-// caller's; attention_decode_static.cu: a fixed array inside the library).
+// The decode attention kernel, its parameter block and its launch by head size, shared by the
+// entry points that differ in where the scratch memory comes from (attention_decode.cu: the
+// caller's; attention_decode_static.cu: a fixed array inside the library) and in whether a window keeps
+// the first keys in sight (attention_decode_kept.cu: the KEEP instances, compiled where a model asks for them).
 #pragma once
 #include "mma_common.cuh"
 #include "tcgen05_common.cuh"      // mbarrier, TMA copies, bounded waits, the tensor-map encoder
@@ -63,7 +64,7 @@ __device__ __forceinline__ uint32_t swz_tile_off(int row, int chunk) {
 // blocks than fit beside one another it is the faster way (128 requests x 512 keys 20.6 -> 14.9 us,
 // 256 x 512 34.4 -> 29.2 us, 256 x 2048 101 -> 96 us = 5.6 TB/s); where a block walks a long part
 // alone it is not (64 x 2048: 40.0 -> 42.9 us), so the caller chooses (ops.decode_uses_tma).
-template <int D, int NSTAGE, bool TMA>
+template <int D, int NSTAGE, bool TMA, bool KEEP>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const DecodeParams p) {
@@ -112,7 +113,7 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // this block's part of the context: the range [lo, ctx) cut into `splits` parts of whole tiles
     const int first_key = mask_first_key(ctx - 1, p.window);      // sliding window, or the start of the query's block of positions
     const int lo = first_key & ~(DEC_TILE - 1);
-    const int kept = mask_kept_tiles(p.keep, lo, DEC_TILE);       // tiles of kept keys in front of the window's
+    const int kept = KEEP ? mask_kept_tiles(p.keep, lo, DEC_TILE) : 0;       // tiles of kept keys in front of the window's
     const int tiles_total = kept + (ctx - lo + DEC_TILE - 1) / DEC_TILE;
     // The grid is laid out for the longest context the launch may meet; a row is cut into as many parts as
     // its own length pays for (scratch merge only: the blocks of a cluster all take part in its barriers).
@@ -163,7 +164,7 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const int* table = p.block_tables + (int64_t)row * p.table_stride;
     // (A part may hold kept tiles and tiles of the window: the pages of its kept tiles come first in the list.  Entry i is
     // the table's entry i + kept_page0 or i + page0.)
-    const int kept_mine = max(0, min(kept - tile0, ntiles));
+    const int kept_mine = KEEP ? max(0, min(kept - tile0, ntiles)) : 0;
     const int kept_page0 = (tile0 * DEC_TILE) >> p.page_shift;
     const int kept_pages = kept_mine > 0 ? (((tile0 + kept_mine) * DEC_TILE - 1) >> p.page_shift) - kept_page0 + 1 : 0;
     const int rest = ntiles - kept_mine, first_page = rest > 0 ? tile_key(kept_mine) >> p.page_shift : 0, page0 = first_page - kept_pages;
@@ -337,7 +338,7 @@ decode_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                     }
                     if (!whole) {
                         const int key = key0 + n * 8 + tq * 2 + (i & 1);
-                        if (!(key < ctx && (key >= first_key || key < p.keep))) v = -INFINITY;
+                        if (!(key < ctx && (key >= first_key || (KEEP && key < p.keep)))) v = -INFINITY;
                     }
                     s[n][i] = v;
                     mx[i >> 1] = fmaxf(mx[i >> 1], v);
@@ -556,7 +557,7 @@ static int make_decode_map(CUtensorMap* map, const void* ptr, uint64_t rows, int
     return r == CUDA_SUCCESS ? 0 : 1000 + (int)r;
 }
 
-template <int D, int NSTAGE, bool TMA>
+template <int D, int NSTAGE, bool TMA, bool KEEP>
 static int launch_decode_stages(const DecodeParams& p, const DecodeMaps& maps, int num_rows, cudaStream_t stream) {
     // at least the four-warp merge buffer (4 x 16 x D float32) must fit
     size_t smem = TMA ? (size_t)NSTAGE * 2 * ((D + 63) / 64) * 8192 + 1024 : (size_t)NSTAGE * 2 * DEC_TILE * (D + 8) * sizeof(bf16);
@@ -565,35 +566,36 @@ static int launch_decode_stages(const DecodeParams& p, const DecodeMaps& maps, i
     DecodeParams pp = p;
     pp.recv_offset = (uint32_t)((smem + 15) & ~size_t(15));
     if (p.cluster) smem = pp.recv_offset + (16 * (D / 4) + 8) * sizeof(float4) + 8 * 16 * sizeof(float);
-    cudaError_t e = cudaFuncSetAttribute(decode_attention_kernel<D, NSTAGE, TMA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(decode_attention_kernel<D, NSTAGE, TMA, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     const dim3 grid(p.splits, p.num_kv_heads * p.chunks, num_rows);
     const dim3 cluster(p.cluster ? p.splits : 1, 1, 1);
-    return launch_kernel_cluster(decode_attention_kernel<D, NSTAGE, TMA>, grid, dim3(DEC_WARPS * 32), smem, stream, cluster,
+    return launch_kernel_cluster(decode_attention_kernel<D, NSTAGE, TMA, KEEP>, grid, dim3(DEC_WARPS * 32), smem, stream, cluster,
                                  maps.k, maps.v, pp);
 }
 
 // Tiles in flight per block.  Few tiles per block (short contexts, many splits): two stages, so that
 // more blocks share an SM and hide one another's latencies.  Many tiles per block: a deeper ring.
-template <int D, bool TMA>
+template <int D, bool TMA, bool KEEP>
 static int launch_decode_tma(const DecodeParams& p, const DecodeMaps& maps, int num_rows, cudaStream_t stream) {
-    if (p.stages <= 2) return launch_decode_stages<D, 2, TMA>(p, maps, num_rows, stream);
-    if (p.stages == 3 || D > 64) return launch_decode_stages<D, 3, TMA>(p, maps, num_rows, stream);
-    return launch_decode_stages<D, 4, TMA>(p, maps, num_rows, stream);
+    if (p.stages <= 2) return launch_decode_stages<D, 2, TMA, KEEP>(p, maps, num_rows, stream);
+    if (p.stages == 3 || D > 64) return launch_decode_stages<D, 3, TMA, KEEP>(p, maps, num_rows, stream);
+    return launch_decode_stages<D, 4, TMA, KEEP>(p, maps, num_rows, stream);
 }
 
-template <int D>
+template <int D, bool KEEP>
 static int launch_decode(const DecodeParams& p, const DecodeMaps& maps, int num_rows, cudaStream_t stream) {
     if constexpr (D == 64 || D == 128) {
-        if (maps.use) return launch_decode_tma<D, true>(p, maps, num_rows, stream);
+        if (maps.use) return launch_decode_tma<D, true, KEEP>(p, maps, num_rows, stream);
     }
-    return launch_decode_tma<D, false>(p, maps, num_rows, stream);
+    return launch_decode_tma<D, false, KEEP>(p, maps, num_rows, stream);
 }
 
 
 // Checks the sizes, fills the parameter block and launches.  With splits > 1 and all three scratch
 // pointers null, the splits (2, 4 or 8) form a thread-block cluster and merge through distributed
 // shared memory; with scratch given, any number of splits merges through it.
+template <bool KEEP>
 static int decode_attention_launch(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
                                    const int* block_tables, int table_stride, const int* row_q_start,
                                    const int* row_q_len, const int* row_ctx_len, int num_rows, void* out,
@@ -620,7 +622,7 @@ static int decode_attention_launch(const void* q, int64_t q_stride, const void* 
     p.num_heads = num_heads; p.num_kv_heads = num_kv_heads; p.page_size = page_size;
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
-    p.window = window; p.keep = keep > 0 ? keep : 0; p.splits = splits; p.cluster = cluster ? 1 : 0;
+    p.window = window; p.keep = KEEP && window && keep > 0 ? keep : 0; p.splits = splits; p.cluster = cluster ? 1 : 0;
     p.stages = stages > 0 ? stages : 4;
     p.min_part_tiles = min_part_tiles > 0 ? min_part_tiles : 0;
     const int G = num_heads / num_kv_heads;
@@ -649,14 +651,14 @@ static int decode_attention_launch(const void* q, int64_t q_stride, const void* 
         p.error = g_error_dev;
     }
     switch (head_dim) {
-        case 16: return launch_decode<16>(p, maps, num_rows, stream);
-        case 32: return launch_decode<32>(p, maps, num_rows, stream);
-        case 48: return launch_decode<48>(p, maps, num_rows, stream);
-        case 64: return launch_decode<64>(p, maps, num_rows, stream);
-        case 80: return launch_decode<80>(p, maps, num_rows, stream);
-        case 96: return launch_decode<96>(p, maps, num_rows, stream);
-        case 112: return launch_decode<112>(p, maps, num_rows, stream);
-        case 128: return launch_decode<128>(p, maps, num_rows, stream);
+        case 16: return launch_decode<16, KEEP>(p, maps, num_rows, stream);
+        case 32: return launch_decode<32, KEEP>(p, maps, num_rows, stream);
+        case 48: return launch_decode<48, KEEP>(p, maps, num_rows, stream);
+        case 64: return launch_decode<64, KEEP>(p, maps, num_rows, stream);
+        case 80: return launch_decode<80, KEEP>(p, maps, num_rows, stream);
+        case 96: return launch_decode<96, KEEP>(p, maps, num_rows, stream);
+        case 112: return launch_decode<112, KEEP>(p, maps, num_rows, stream);
+        case 128: return launch_decode<128, KEEP>(p, maps, num_rows, stream);
     }
     return MIE_ERR_BAD_ARG;
 }

@@ -75,7 +75,7 @@ extern "C" int mie_decode_attention_static(const void* q, int64_t q_stride, cons
         const cudaError_t e = cudaMemsetAsync(counters, 0, (size_t)units * sizeof(int), stream);
         if (e != cudaSuccess) { snprintf(g_error, sizeof g_error, "cudaMemsetAsync failed: %s", cudaGetErrorString(e)); return (int)e; }
     }
-    const int rc = decode_attention_launch(q, q_stride, k_cache, v_cache, block_tables, table_stride, row_q_start,
+    const int rc = decode_attention_launch<false>(q, q_stride, k_cache, v_cache, block_tables, table_stride, row_q_start,
                                            row_q_len, row_ctx_len, num_rows, out, num_heads, num_kv_heads, head_dim,
                                            page_size, scale, window, splits, part_o, part_lse, counters, stream);
     if (rc < 0) snprintf(g_error, sizeof g_error, "the decode kernel refused the sizes (code %d): head_dim a multiple of 16 up to %d, "

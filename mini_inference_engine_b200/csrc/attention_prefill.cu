@@ -38,8 +38,8 @@ struct PrefillParams {
 };
 
 // MODS: the instance for scores that are modified before the softmax (a cap, a bias by distance: ScoreMods) and for a sink; the
-// plain instance tests nothing per score.
-template <int D, bool MODS>
+// plain instance tests nothing per score.  KEEP: the instance for a window or block that keeps the first keys in sight (p.keep).
+template <int D, bool MODS, bool KEEP>
 __global__ void __launch_bounds__(PRE_WARPS * 32)
 prefill_attention_kernel(const PrefillParams p) {
     constexpr int DP = D + 8;
@@ -75,7 +75,7 @@ prefill_attention_kernel(const PrefillParams p) {
     const int k_hi = pos0 + nq;                                     // one past the last key any query reads
     const int k_lo = mask_first_key(pos0, p.window);
     const int kbeg = k_lo & ~(PRE_BN - 1);
-    const int kept = mask_kept_tiles(p.keep, kbeg, PRE_BN);         // tiles of kept keys in front of the window's
+    const int kept = KEEP ? mask_kept_tiles(p.keep, kbeg, PRE_BN) : 0;         // tiles of kept keys in front of the window's
     const int ntiles = kept + (k_hi - kbeg + PRE_BN - 1) / PRE_BN;
     auto tile_key = [&](int t) { return t < kept ? t * PRE_BN : kbeg + (t - kept) * PRE_BN; };
 
@@ -91,6 +91,7 @@ prefill_attention_kernel(const PrefillParams p) {
                                      p.q + (int64_t)(q_start + q0 + r) * p.q_stride + (int64_t)head * D + c) : 0u;
         }
     const int qpos[2] = {pos0 + wq + quad, pos0 + wq + quad + 8};
+    const int qfirst[2] = {mask_first_key(qpos[0], p.window), mask_first_key(qpos[1], p.window)};     // once a row: a block's start is a division
     const bool warp_has_rows = wq < nq;
 
     float o[NBLK][4];
@@ -123,7 +124,7 @@ prefill_attention_kernel(const PrefillParams p) {
         for (int idx = threadIdx.x; idx < PRE_BN * CHUNKS_PER_ROW; idx += PRE_WARPS * 32) {
             const int r = idx / CHUNKS_PER_ROW, c = (idx - r * CHUNKS_PER_ROW) * 8;
             const int key = k0 + r;
-            if ((key >= k_lo || key < p.keep) && key < k_hi) {
+            if ((key >= k_lo || (KEEP && key < p.keep)) && key < k_hi) {
                 const int e = key >> p.page_shift, pi = e - page0;
                 const int page = pi < PRE_PAGE_SLOTS ? s_pages[pi] : checked_page(table[e], p.check_pages, p.report, MIE_K_ATTENTION_PREFILL, e);
                 const int64_t src = (((int64_t)page * p.num_kv_heads + kvh) * p.page_size + (key & (p.page_size - 1))) * D + c;
@@ -176,8 +177,7 @@ prefill_attention_kernel(const PrefillParams p) {
                         v = mod_score<true>(s[n][i] * p.scale, p.mods, head, p.num_heads, qpos[i >> 1] - (key0 + n * 8 + tq * 2 + (i & 1))) * 1.4426950408889634f;
                     if (need_mask) {
                         const int key = key0 + n * 8 + tq * 2 + (i & 1);
-                        const int qp = qpos[i >> 1];
-                        const bool ok = mask_reads(qp, key, p.window, p.keep);
+                        const bool ok = key <= qpos[i >> 1] && (key >= qfirst[i >> 1] || (KEEP && key < p.keep));
                         v = ok ? v : -INFINITY;
                     }
                     s[n][i] = v;
@@ -252,18 +252,19 @@ prefill_attention_kernel(const PrefillParams p) {
     }
 }
 
-template <int D, bool MODS>
+template <int D, bool MODS, bool KEEP>
 static int launch_prefill_as(const PrefillParams& p, int work_tokens, int work_rows, cudaStream_t stream) {
     const size_t smem = (size_t)2 * 2 * PRE_BN * (D + 8) * sizeof(bf16);
-    cudaError_t e = cudaFuncSetAttribute(prefill_attention_kernel<D, MODS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(prefill_attention_kernel<D, MODS, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     const dim3 grid((work_tokens + PRE_BM - 1) / PRE_BM + work_rows, p.num_heads);     // tiles <= tokens / 64 + rows
-    return launch_kernel(prefill_attention_kernel<D, MODS>, grid, dim3(PRE_WARPS * 32), smem, stream, p);
+    return launch_kernel(prefill_attention_kernel<D, MODS, KEEP>, grid, dim3(PRE_WARPS * 32), smem, stream, p);
 }
 template <int D>
 static int launch_prefill(const PrefillParams& p, int work_tokens, int work_rows, cudaStream_t stream) {
-    return (p.modded || p.mods.sink) ? launch_prefill_as<D, true>(p, work_tokens, work_rows, stream)
-                                     : launch_prefill_as<D, false>(p, work_tokens, work_rows, stream);
+    if (p.keep) return launch_prefill_as<D, true, true>(p, work_tokens, work_rows, stream);
+    return (p.modded || p.mods.sink) ? launch_prefill_as<D, true, false>(p, work_tokens, work_rows, stream)
+                                     : launch_prefill_as<D, false, false>(p, work_tokens, work_rows, stream);
 }
 
 // Rows with fewer than `min_q_len` new tokens are skipped (the decode kernel serves single tokens).  work_rows /
@@ -291,7 +292,7 @@ extern "C" int mie_prefill_attention(const void* q, int64_t q_stride, const void
     p.num_heads = num_heads; p.num_kv_heads = num_kv_heads; p.page_size = page_size;
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
-    p.window = window; p.keep = keep > 0 ? keep : 0; p.min_q_len = min_q_len;
+    p.window = window; p.keep = window && keep > 0 ? keep : 0; p.min_q_len = min_q_len;
     p.scale_log2e = scale * 1.4426950408889634f;
     if (dist_bias && dist_len <= 0) return MIE_ERR_BAD_ARG;
     p.scale = scale;

@@ -105,8 +105,9 @@ __device__ __forceinline__ float ex2_approx(float x) {
 
 // MODS: what scores pass between the product and the softmax (ScoreMods): bit 0 a cap, bit 1 a bias by distance; an instance
 // for each combination, so that the plain softmax keeps its instruction count and the others test nothing per element.  A sink
-// joins the sum in every instance (it costs a term at a row's start).
-template <int D, int MODS>
+// joins the sum in every instance (it costs a term at a row's start).  KEEP: the instance for a window or block that keeps the
+// first keys in sight (p.keep).
+template <int D, int MODS, bool KEEP>
 __global__ void __launch_bounds__(FA_THREADS, MODS ? 1 : 2)       // two blocks per SM: at most 168 registers (the instance with
                                                                   // modified scores needs more and takes an SM alone)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv activation [tokens, q_stride], box {64, 128}
@@ -203,7 +204,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
             g.k_hi = g.pos0 + g.nq;                              // one past the last key any query here reads
             g.k_lo = mask_first_key(g.pos0, p.window);
             g.kbeg = g.k_lo & ~(FA_BN - 1);
-            g.kept = mask_kept_tiles(p.keep, g.kbeg, FA_BN);     // tiles of kept keys in front of the window's
+            g.kept = KEEP ? mask_kept_tiles(p.keep, g.kbeg, FA_BN) : 0;     // tiles of kept keys in front of the window's
             g.ntiles = u < nsub ? g.kept + (g.k_hi - g.kbeg + FA_BN - 1) / FA_BN : 0;
         }
         const int nA = sb[0].ntiles, G = nA + sb[1].ntiles;      // key tiles of the first query tile, and of both
@@ -350,7 +351,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
             for (int u = 0; u < nsub && ok; ++u) {                 // one query tile after the other
                 const int q0 = sb[u].q0, pos0 = sb[u].pos0, nq = sb[u].nq, k_lo = sb[u].k_lo, kbeg = sb[u].kbeg, kept = sb[u].kept, ntiles = sb[u].ntiles;
                 const int g0 = u ? nA : 0;                             // key tiles counted through both query tiles
-                const int qpos = pos0 + r;
+                const int qpos = pos0 + r, row_lo = mask_first_key(qpos, p.window);
                 float m_run = -INFINITY, l_run = 0.f;
                 if (p.mods.sink) { m_run = p.mods.sink[head] * 1.4426950408889634f; l_run = 1.f; }      // the sink: a term with no value
                 // a modified score in base 2, from the raw product and the key's position
@@ -371,7 +372,16 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                     tc_fence_after();
                     const int key0 = t < kept ? t * FA_BN : kbeg + (t - kept) * FA_BN;
                     // masks are needed only where the tile touches the diagonal, the window's edge or the range's start
-                    const bool need_mask = key0 + FA_BN - 1 > pos0 || key0 < k_lo || (p.window != 0 && key0 < mask_first_key(pos0 + FA_BM - 1, p.window));
+                    bool need_mask = key0 + FA_BN - 1 > pos0 || key0 < k_lo || (p.window != 0 && key0 < mask_first_key(pos0 + FA_BM - 1, p.window));
+                    // A key is read if lo <= key <= hi or, with kept keys, if it is below `also`: a tile in front of the window's holds kept
+                    // keys only (earlier than every query), a tile of the window may begin with some.  The bounds are the row's, worked out
+                    // once: inside the loops over elements the mask's rule (a block's start is a division) costs more than all else there.
+                    int lo = row_lo, hi = qpos, also = p.keep;
+                    if (KEEP) {
+                        const bool front = t < kept;
+                        if (front) { lo = 0; hi = p.keep - 1; also = 0; }
+                        if (front) need_mask = key0 + FA_BN > p.keep;
+                    }
                     // The row of S comes out of TMEM in four chunks of 32 columns; the load of the next chunk is
                     // in flight while the current one is worked on.
                     auto for_each_chunk = [&](auto&& body) {
@@ -389,7 +399,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                         tmem_ld_wait(cb);
                         body(3, cb);
                     };
-                    auto masked = [&](int key) { return !mask_reads(qpos, key, p.window, p.keep); };
+                    auto masked = [&](int key) {
+                        return key > hi || (key < lo && (!KEEP || key >= also));
+                    };
                     // Reference point of the exponent.  Reading S once per tile is what matters here (TMEM
                     // loads are the slowest part of the step), so the running max is not recomputed up front:
                     // P is formed against the running max as it stands, the row's true max is found on the
@@ -764,7 +776,7 @@ prefill_attention_pp_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (u < nsub) {
                 const int q0 = u ? sb[1].q0 : sb[0].q0, pos0 = u ? sb[1].pos0 : sb[0].pos0, nq = u ? sb[1].nq : sb[0].nq;
                 const int k_lo = u ? k_lo1 : k_lo0;
-                const int qpos = pos0 + r;
+                const int qpos = pos0 + r, row_lo = mask_first_key(qpos, p.window);
                 float m_run = -INFINITY, l_run = 0.f;
                 int used = 0;                                      // key tiles this group has taken
                 // The two groups take turns at the exponent unit: with both in it at once each takes twice as long
@@ -793,7 +805,7 @@ prefill_attention_pp_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     __syncwarp();
                     if (lane == 0) mbar_arrive(&s_free[u]);
                     if (q == 2 && lane == 0) { PP_STAMP(u, j, 1); }
-                    auto masked = [&](int key) { return !(key <= qpos && key >= mask_first_key(qpos, p.window)); };
+                    auto masked = [&](int key) { return key > qpos || key < row_lo; };
                     if (need_mask) {                               // masked entries become -inf once, here
 #pragma unroll
                         for (int i = 0; i < 128; ++i) if (masked(key0 + i)) sv[i] = __float_as_uint(-INFINITY);
@@ -929,11 +941,11 @@ static int make_map_2d(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_
 
 static int g_fa_pp_mode = -1;
 
-template <int D, int MODS>
+template <int D, int MODS, bool KEEP>
 static int launch_fa(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FaParams& p, int work_tokens,
                      int work_rows, cudaStream_t stream) {
     const size_t smem = (size_t)(D / 64) * 128 * 64 * 2 * 6 + 1024;     // 2 x Q + 2 x (K + V)
-    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, MODS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, MODS, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     // tiles <= tokens / 128 + rows (of the rows that this kernel serves, where the caller knows them); a block takes
     // one tile, or a pair of them (at most (tiles + rows) / 2 pairs) once the tiles of all heads are more than the
@@ -942,7 +954,7 @@ static int launch_fa(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
     FaParams pp = p;
     pp.pair = (int64_t)tiles * p.num_heads > (int64_t)device_sm_count() * (D == 64 ? 2 : 1);
     const dim3 grid(pp.pair ? (tiles + work_rows + 1) / 2 : tiles, p.num_heads);
-    return launch_kernel(prefill_attention_tc_kernel<D, MODS>, grid, dim3(FA_THREADS), smem, stream, mq, mk, mv, pp);
+    return launch_kernel(prefill_attention_tc_kernel<D, MODS, KEEP>, grid, dim3(FA_THREADS), smem, stream, mq, mk, mv, pp);
 }
 
 // q: the fused qkv activation [num_tokens, q_stride] bfloat16 (query head h at columns h*D ..), caches
@@ -972,7 +984,7 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
     p.num_heads = num_heads; p.num_kv_heads = num_kv_heads; p.page_size = page_size;
     p.page_shift = 0;
     while ((1 << p.page_shift) < page_size) ++p.page_shift;
-    p.window = window; p.keep = keep > 0 ? keep : 0; p.min_q_len = min_q_len; p.pair = 0;
+    p.window = window; p.keep = window && keep > 0 ? keep : 0; p.min_q_len = min_q_len; p.pair = 0;
     p.scale_log2e = scale * 1.4426950408889634f;
     p.scale = scale;
     p.mods = ScoreMods{softcap, sink, dist_bias, dist_len};
@@ -985,12 +997,15 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
     if ((rc = make_map_2d(&mq, q, (uint64_t)num_tokens, (uint64_t)q_stride, (uint64_t)q_stride, FA_BM))) return rc;
     if ((rc = make_map_2d(&mk, k_cache, cache_rows, (uint64_t)head_dim, (uint64_t)head_dim, box_rows))) return rc;
     if ((rc = make_map_2d(&mv, v_cache, cache_rows, (uint64_t)head_dim, (uint64_t)head_dim, box_rows))) return rc;
-#define FA_MODS(DD) (mods == 1 ? launch_fa<DD, 1>(mq, mk, mv, p, work_tokens, work_rows, stream)                                  \
-                     : mods == 2 ? launch_fa<DD, 2>(mq, mk, mv, p, work_tokens, work_rows, stream)                                \
-                                 : launch_fa<DD, 3>(mq, mk, mv, p, work_tokens, work_rows, stream))
+#define FA_MODS(DD) (mods == 1 ? launch_fa<DD, 1, false>(mq, mk, mv, p, work_tokens, work_rows, stream)                                  \
+                     : mods == 2 ? launch_fa<DD, 2, false>(mq, mk, mv, p, work_tokens, work_rows, stream)                                \
+                                 : launch_fa<DD, 3, false>(mq, mk, mv, p, work_tokens, work_rows, stream))
+    if (mods && p.keep) return MIE_ERR_BAD_ARG;        // kept keys with a cap or a bias: the mma.sync kernel takes those
     if (mods) return head_dim == 64 ? FA_MODS(64) : FA_MODS(128);
 #undef FA_MODS
-    if (head_dim == 64 && !sink && p.keep == 0) {        // (the kernel with two query tiles side by side has no sink and no kept keys)
+    if (p.keep) return head_dim == 64 ? launch_fa<64, 0, true>(mq, mk, mv, p, work_tokens, work_rows, stream)
+                                      : launch_fa<128, 0, true>(mq, mk, mv, p, work_tokens, work_rows, stream);
+    if (head_dim == 64 && !sink) {        // (the kernel with two query tiles side by side has no sink and no kept keys)
         // two query tiles side by side once there are three pairs for every SM (measured, 32 heads, one tile a block
         // against two side by side: 2,048 tokens 45.1 against 48.5 us, 4,096 tokens 143.7 against 142.4 us, 8,192 tokens
         // 496 against 462 us); below that the one-tile blocks, two on an SM, spread a launch over more SMs
@@ -998,10 +1013,10 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
         if ((tiles + 2 * work_rows) / 2 < 65535 &&
             (g_fa_pp_mode == 1 || (g_fa_pp_mode < 0 && tiles * num_heads >= 6 * (int64_t)device_sm_count())))
             return launch_fa_pp(mq, mk, mv, p, work_tokens, work_rows, stream);
-        return launch_fa<64, 0>(mq, mk, mv, p, work_tokens, work_rows, stream);
+        return launch_fa<64, 0, false>(mq, mk, mv, p, work_tokens, work_rows, stream);
     }
-    if (head_dim == 64) return launch_fa<64, 0>(mq, mk, mv, p, work_tokens, work_rows, stream);
-    return launch_fa<128, 0>(mq, mk, mv, p, work_tokens, work_rows, stream);
+    if (head_dim == 64) return launch_fa<64, 0, false>(mq, mk, mv, p, work_tokens, work_rows, stream);
+    return launch_fa<128, 0, false>(mq, mk, mv, p, work_tokens, work_rows, stream);
 }
 
 // Which kernel serves head_dim 64: -1 chooses by the size of the launch (the default), 0 always one query tile a block,

@@ -98,7 +98,9 @@ def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, wi
                              max_ctx=reach, mods=mods, keep=keep)
     if has_prefill:
         # tcgen05 (S and O in tensor memory) for the head sizes it is written for, mma.sync otherwise
-        tc = head_dim in (64, 128) and cache.page_size >= 8 and q_stride % 8 == 0 and _prefill_backend == "tcgen05"
+        # (kept keys with a cap or a bias by distance: mma.sync, the tcgen05 kernel has no instance for them)
+        tc = (head_dim in (64, 128) and cache.page_size >= 8 and q_stride % 8 == 0 and _prefill_backend == "tcgen05"
+              and not (keep and mods is not None and (mods.softcap > 0 or mods.dist_bias is not None)))
         fn = ops.prefill_attention_tc if tc else ops.prefill_attention
         # the rows that are portions, and their tokens: the launch is laid out for those, not for every decoding row
         work = None if kinds is None else (kinds[1], kinds[2])

@@ -32,7 +32,7 @@ COMMON_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--shared", "-Xcompiler", "-fP
                 "-Xcompiler", "-fvisibility=default"]
 
 # every source file of the package; `build_all` compiles all of them
-SOURCES = ("embedding", "norm", "rope_cache", "attention_simt", "attention_decode", "attention_decode_static", "attention_prefill",
+SOURCES = ("embedding", "norm", "rope_cache", "attention_simt", "attention_decode", "attention_decode_kept", "attention_decode_static", "attention_prefill",
            "attention_prefill_tc",
            "activation", "gemm_simt", "gemm_tcgen05", "gemm_chain", "gemm_pair_tc",
            "sampling", "norm_group", "qk_norm_rope", "retention", "linear_recurrence",

@@ -426,7 +426,8 @@ def prefill_attention_tc(q: torch.Tensor, q_stride: int, k_cache, v_cache, block
                          head_dim: int, page_size: int, scale: float, window: int | None = None,
                          min_q_len: int = 2, work=None, mods: ScoreMods | None = None, keep: int = 0) -> torch.Tensor:
     """Causal attention of prompt portions on tcgen05 (S and O in tensor memory, operands by TMA);
-    head_dim 64 or 128.  ``work``: as for ``prefill_attention``."""
+    head_dim 64 or 128.  ``work``: as for ``prefill_attention``.  Kept keys (``keep``) go with a plain score or a sink, not with a cap or
+    a bias."""
     _need(q.dtype == torch.bfloat16 == k_cache.dtype == v_cache.dtype and out.dtype in (torch.bfloat16, torch.float32),
           "prefill attention is bfloat16 (its output bfloat16 or float32)")
     _need(head_dim in (64, 128), f"head_dim {head_dim}: the tcgen05 prefill kernel takes 64 and 128")
@@ -460,7 +461,8 @@ def set_prefill_pairs(mode: int = -1) -> None:
 
 def check_tc_errors() -> None:
     """Raises if a block of a tensor-core kernel gave up a bounded wait (call after a synchronise)."""
-    for name, fn in (("attention_prefill_tc", "mie_prefill_attention_tc"), ("attention_decode", "mie_decode_attention")):
+    for name, fn in (("attention_prefill_tc", "mie_prefill_attention_tc"), ("attention_decode", "mie_decode_attention"),
+                     ("attention_decode_kept", "mie_decode_attention_kept")):
         lib = build._libs.get(name)
         if lib is not None and getattr(lib, fn + "_error")():
             getattr(lib, fn + "_clear_error")()
@@ -645,11 +647,21 @@ def decode_attention(q: torch.Tensor, q_stride: int, k_cache, v_cache, block_tab
         part_o = _workspace(q.device, "decode_part_o", rows * num_heads * splits * head_dim, torch.float32)
         part_lse = _workspace(q.device, "decode_part_lse", rows * num_heads * splits, torch.float32)
         counters = _workspace(q.device, "decode_counters", rows * num_kv_heads * chunks, torch.int32)
+    if keep and window:
+        _need(rope is None, "rotation inside the decode kernel does not go together with kept keys")
+        _check(load("attention_decode_kept").mie_decode_attention_kept(
+            _ptr(q), ctypes.c_int64(q_stride), _ptr(k_cache), _ptr(v_cache), _ptr(block_tables), block_tables.shape[1], _ptr(row_q_start),
+            _ptr(row_q_len), _ptr(row_ctx_len), rows, _ptr(out), num_heads, num_kv_heads, head_dim, page_size, ctypes.c_float(scale),
+            int(window), int(keep), int(splits), _ptr(part_o), _ptr(part_lse), _ptr(counters), int(stages or 0),
+            ctypes.c_int64(k_cache.shape[0] if tma else 0), ctypes.c_int64(k_cache.shape[0]),
+            int(min_part_tiles if merge == "scratch" else 0), int(out.dtype == torch.float32), *(mods or _NO_MODS).args(num_heads),
+            _stream()), "decode_attention with kept keys")
+        return out
     lib = load("attention_decode")
     _check(lib.mie_decode_attention(_ptr(q), ctypes.c_int64(q_stride), _ptr(k_cache), _ptr(v_cache),
                                     _ptr(block_tables), block_tables.shape[1], _ptr(row_q_start), _ptr(row_q_len),
                                     _ptr(row_ctx_len), rows, _ptr(out), num_heads, num_kv_heads, head_dim,
-                                    page_size, ctypes.c_float(scale), int(window or 0), int(keep), int(splits),
+                                    page_size, ctypes.c_float(scale), int(window or 0), int(splits),
                                     _ptr(part_o), _ptr(part_lse), _ptr(counters), int(stages or 0),
                                     ctypes.c_int64(k_cache.shape[0] if tma else 0), ctypes.c_int64(k_cache.shape[0]),
                                     int(min_part_tiles if merge == "scratch" else 0),

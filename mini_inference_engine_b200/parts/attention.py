@@ -220,11 +220,7 @@ class GatedAttention(Mixer):
 
     def kernel_sources(self):
         names = self.rt.product_sources(self.w_in, self.w_o) | {"qk_norm_rope", "activation"}
-        if self.rt.dtype == torch.float32 or self.padded > 128:
-            names.add("attention_simt")
-        else:
-            names |= {"attention_decode", "attention_prefill_tc" if self.padded in (64, 128) else "attention_prefill"}
-        return names
+        return names | _attention_sources(self.rt, self.padded, self.keep_first)
 
     def forward(self, x, ctx, cache):
         from ..kernels import ops
@@ -266,10 +262,10 @@ def _padded_rows(parts, multiple: int = 8):
     return w, n
 
 
-def _attention_sources(rt, padded: int) -> set:
+def _attention_sources(rt, padded: int, keep: int = 0) -> set:
     if rt.dtype == torch.float32 or padded > 128:
         return {"attention_simt"}
-    return {"attention_decode", "attention_prefill_tc" if padded in (64, 128) else "attention_prefill"}
+    return {"attention_decode_kept" if keep else "attention_decode", "attention_prefill_tc" if padded in (64, 128) else "attention_prefill"}
 
 
 class DifferentialAttention(Mixer):
