@@ -134,7 +134,7 @@ def test_configurations_that_are_refused(edit, word):
 
 def test_rotary_frequencies_linear_and_yarn():
     from mini_inference_engine_b200.parts.rope import rotary_frequencies, rotary_gain
-    cases = [(16, 2.5e5, dict(factor=4.0, original=512, fast=32.0, slow=1.0)), (64, 1e4, dict(factor=40.0, original=4096, fast=32.0, slow=1.0)),
+    cases = [(24, 1.5e5, dict(factor=4.0, original=700, fast=24.0, slow=1.0)), (64, 1e4, dict(factor=40.0, original=4096, fast=32.0, slow=1.0)),
              (8, 50.0, dict(factor=1.0, original=64, fast=4.0, slow=2.0)),
              (32, 1e6, dict(factor=8.0, original=100000, fast=500.0, slow=0.01)),       # the ramp's ends lie beyond both ends of the pairs
              (12, 1e3, dict(factor=2.0, original=30, fast=1.5, slow=1.5))]             # both ends on one pair
@@ -146,7 +146,7 @@ def test_rotary_frequencies_linear_and_yarn():
     assert torch.equal(rotary_frequencies(10, 300.0, dict(kind="linear", factor=2.5)), torch.tensor(pr.linear_speeds(10, 300.0, 2.5), dtype=torch.float32))
     assert rotary_gain(dict(kind="linear", factor=2.5)) == rotary_gain(None) == 1.0
     # a mixture: some pairs keep their frequency, some get f / factor, some lie between
-    f, s = rotary_frequencies(16, 2.5e5), rotary_frequencies(16, 2.5e5, dict(cases[0][2], kind="yarn"))
+    f, s = rotary_frequencies(24, 1.5e5), rotary_frequencies(24, 1.5e5, dict(cases[0][2], kind="yarn"))
     ratio = (s / f).tolist()
     assert ratio[0] == 1.0 and ratio[-1] == pytest.approx(0.25) and any(0.26 < r < 0.99 for r in ratio)
     with pytest.raises(ValueError):

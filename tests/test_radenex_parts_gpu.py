@@ -329,9 +329,9 @@ def latent(heads, dim, rot_dim, vdim, kv_rank, scale, base, scaling, hidden=40):
 
 
 YARN = dict(factor=6.0, original=40, fast=8.0, slow=1.0)
-LATENT = [latent(3, 16, 8, 32, 24, 0.3, 500.0, YARN), latent(1, 48, 16, 64, 16, 0.15, 1e4, dict(factor=1.0, original=512, fast=32.0, slow=1.0)),
+LATENT = [latent(3, 16, 8, 32, 24, 0.3, 500.0, YARN), latent(1, 48, 16, 64, 16, 0.15, 1e4, dict(factor=1.0, original=300, fast=20.0, slow=1.0)),
           latent(2, 96, 32, 128, 40, 0.1, 3e4, dict(factor=32.0, original=30, fast=2.0, slow=0.5)), latent(5, 10, 6, 20, 9, 0.4, 100.0, YARN),
-          latent(2, 120, 24, 40, 32, 0.1, 1e4, YARN), latent(4, 16, 48, 16, 48, 0.2, 1e3, None), latent(8, 64, 64, 48, 128, 0.1, 2e5, YARN, hidden=64)]
+          latent(2, 120, 24, 40, 32, 0.1, 1e4, YARN), latent(4, 16, 48, 16, 48, 0.2, 1e3, None), latent(7, 56, 56, 40, 112, 0.1, 2e5, YARN, hidden=72)]
 
 
 @pytest.mark.parametrize("dt", DTYPES)
