@@ -4,7 +4,8 @@ state slots per layer.
 Layers are grouped by need (see ``CacheLayout``); every group has its own page id space, so a
 layer's tensors have as many pages as its group's pool.  A layer's pages are one tensor
 ``[2 (k, v), pages, kv_heads, page_size, head_dim]``: all slots of one (page, head) are contiguous,
-so a kernel that works per kv head reads a page as one ``page_size x head_dim`` box.  (The
+so a kernel that works per kv head reads a page as one ``page_size x head_dim`` box.  (A layer whose keys serve as values
+has ``[1, ...]``, and k and v are the same pages.)  (The
 reference has one tensor ``[L, 2, NB, 16, H_kv, D]`` for all layers, inference_engine/model.py:39-53.)
 Page 0 and state slot 0 are scratch: padding rows of a captured decode step read and write them.
 """
@@ -70,7 +71,7 @@ class CacheLayout:
 
     def bytes_per_page(self, group: int, page_size: int, dtype: torch.dtype) -> int:
         el = torch.empty((), dtype=dtype).element_size()
-        return sum(2 * page_size * n.num_kv_heads * n.head_dim * el for g, n in self.kv.values() if g == group)
+        return sum((1 if n.shared else 2) * page_size * n.num_kv_heads * n.head_dim * el for g, n in self.kv.values() if g == group)
 
     def bytes_per_state_slot(self) -> int:
         total = 0
@@ -91,7 +92,7 @@ class CacheStorage:
         self.num_state_slots = num_state_slots
         self.kv = {}
         for layer, (g, need) in layout.kv.items():
-            self.kv[layer] = torch.zeros(2, self.num_pages[g], need.num_kv_heads, page_size, need.head_dim,
+            self.kv[layer] = torch.zeros(1 if need.shared else 2, self.num_pages[g], need.num_kv_heads, page_size, need.head_dim,
                                          dtype=dtype, device=device)
         self.state = {layer: torch.zeros((num_state_slots + 1,) + tuple(n.shape), dtype=n.dtype, device=device)
                       for layer, n in layout.state.items()}
@@ -103,7 +104,7 @@ class CacheStorage:
             return lc
         if owner in self.kv:
             lc.group = self.layout.kv[owner][0]
-            lc.k, lc.v = self.kv[owner][0], self.kv[owner][1]
+            lc.k, lc.v = self.kv[owner][0], self.kv[owner][-1]
         if owner in self.state:
             lc.state = self.state[owner]
         return lc

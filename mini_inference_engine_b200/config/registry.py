@@ -5,6 +5,7 @@ The reference has no registry (inference_engine/engine.py:44 builds Llama for an
 from __future__ import annotations
 
 from .getizen_config import GetizenConfig
+from .karopel_config import KaropelConfig
 from .kebudra_config import KebudraConfig
 from .luluzen_config import LuluzenConfig
 from .radenex_config import RadenexConfig
@@ -48,6 +49,7 @@ register_architecture("Kebudra", KebudraConfig)
 register_architecture("Serotar", SerotarConfig)
 register_architecture("Luluzen", LuluzenConfig)
 register_architecture("Radenex", RadenexConfig)
+register_architecture("Karopel", KaropelConfig)
 
 
 def preset_names() -> list[str]:

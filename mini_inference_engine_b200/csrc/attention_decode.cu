@@ -49,8 +49,8 @@ extern "C" int mie_decode_attention(const void* q, int64_t q_stride, const void*
                                     int window, int splits, float* part_o, float* part_lse, int* counters,
                                     int stages, int64_t num_pages, int64_t check_pages, int min_part_tiles,
                                     const float* cos_t, const float* sin_t, int max_pos, int out_f32, float softcap,
-                                    const float* sink, const float* dist_bias, int dist_len, cudaStream_t stream) {
-    const ScoreMods mods{softcap, sink, dist_bias, dist_len};
+                                    const float* sink, const float* dist_bias, int dist_len, const float* slope, cudaStream_t stream) {
+    const ScoreMods mods{softcap, sink, dist_bias, dist_len, slope};
     return decode_attention_launch<false>(q, q_stride, k_cache, v_cache, block_tables, table_stride, row_q_start, row_q_len,
                                    row_ctx_len, num_rows, out, num_heads, num_kv_heads, head_dim, page_size, scale,
                                    window, splits, part_o, part_lse, counters, stream, stages, num_pages, check_pages,

@@ -629,9 +629,9 @@ static int decode_attention_launch(const void* q, int64_t q_stride, const void* 
     p.chunks = (G + 15) / 16;
     p.scale_log2e = scale * 1.4426950408889634f;
     p.scale = scale;
-    p.mods = mods ? *mods : ScoreMods{0.f, nullptr, nullptr, 0};
+    p.mods = mods ? *mods : ScoreMods{0.f, nullptr, nullptr, 0, nullptr};
     if (p.mods.dist_bias && p.mods.dist_len <= 0) return MIE_ERR_BAD_ARG;
-    p.modded = p.mods.softcap > 0.f || p.mods.dist_bias != nullptr;
+    p.modded = p.mods.softcap > 0.f || p.mods.dist_bias != nullptr || p.mods.slope != nullptr;
     p.check_pages = check_pages; p.report = report;
     if ((cos_t != nullptr) != (sin_t != nullptr) || (cos_t && (head_dim % 32 || max_pos <= 0))) return MIE_ERR_BAD_ARG;
     p.cos_t = cos_t; p.sin_t = sin_t; p.max_pos = max_pos;

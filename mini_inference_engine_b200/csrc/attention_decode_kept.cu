@@ -10,9 +10,9 @@ extern "C" int mie_decode_attention_kept(const void* q, int64_t q_stride, const 
                                          int num_heads, int num_kv_heads, int head_dim, int page_size, float scale,
                                          int window, int keep, int splits, float* part_o, float* part_lse, int* counters,
                                          int stages, int64_t num_pages, int64_t check_pages, int min_part_tiles, int out_f32,
-                                         float softcap, const float* sink, const float* dist_bias, int dist_len, cudaStream_t stream) {
+                                         float softcap, const float* sink, const float* dist_bias, int dist_len, const float* slope, cudaStream_t stream) {
     if (window == 0 || keep <= 0) return MIE_ERR_BAD_ARG;
-    const ScoreMods mods{softcap, sink, dist_bias, dist_len};
+    const ScoreMods mods{softcap, sink, dist_bias, dist_len, slope};
     return decode_attention_launch<true>(q, q_stride, k_cache, v_cache, block_tables, table_stride, row_q_start, row_q_len,
                                          row_ctx_len, num_rows, out, num_heads, num_kv_heads, head_dim, page_size, scale,
                                          window, splits, part_o, part_lse, counters, stream, stages, num_pages, check_pages,

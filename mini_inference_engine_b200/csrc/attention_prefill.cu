@@ -276,7 +276,7 @@ extern "C" int mie_prefill_attention(const void* q, int64_t q_stride, const void
                                      void* out, int num_heads, int num_kv_heads, int head_dim, int page_size,
                                      float scale, int window, int keep, int min_q_len, long long num_pages, int work_rows,
                                      int work_tokens, int out_f32, float softcap, const float* sink, const float* dist_bias,
-                                     int dist_len, cudaStream_t stream) {
+                                     int dist_len, const float* slope, cudaStream_t stream) {
     if (num_rows <= 0 || num_tokens <= 0) return 0;
     if (work_rows <= 0 || work_tokens <= 0 || work_rows > num_rows || work_tokens > num_tokens) { work_rows = num_rows; work_tokens = num_tokens; }
     if (head_dim < 16 || head_dim > PRE_MAX_D || head_dim % 16) return MIE_ERR_BAD_ARG;
@@ -296,8 +296,8 @@ extern "C" int mie_prefill_attention(const void* q, int64_t q_stride, const void
     p.scale_log2e = scale * 1.4426950408889634f;
     if (dist_bias && dist_len <= 0) return MIE_ERR_BAD_ARG;
     p.scale = scale;
-    p.mods = ScoreMods{softcap, sink, dist_bias, dist_len};
-    p.modded = softcap > 0.f || dist_bias != nullptr;
+    p.mods = ScoreMods{softcap, sink, dist_bias, dist_len, slope};
+    p.modded = softcap > 0.f || dist_bias != nullptr || slope != nullptr;
     p.check_pages = num_pages > 0 ? (int64_t)num_pages : ((int64_t)1 << 40); p.report = g_range_report;
     switch (head_dim) {
         case 16: return launch_prefill<16>(p, work_tokens, work_rows, stream);

@@ -103,13 +103,13 @@ __device__ __forceinline__ float ex2_approx(float x) {
     return y;
 }
 
-// MODS: what scores pass between the product and the softmax (ScoreMods): bit 0 a cap, bit 1 a bias by distance; an instance
-// for each combination, so that the plain softmax keeps its instruction count and the others test nothing per element.  A sink
+// MODS: what scores pass between the product and the softmax (ScoreMods): bit 0 a cap, bit 1 a bias by distance, bit 2
+// a slope by distance (alone); an instance for each combination, so that the plain softmax keeps its instruction count and the others test nothing per element.  A sink
 // joins the sum in every instance (it costs a term at a row's start).  KEEP: the instance for a window or block that keeps the
 // first keys in sight (p.keep).
 template <int D, int MODS, bool KEEP>
-__global__ void __launch_bounds__(FA_THREADS, MODS ? 1 : 2)       // two blocks per SM: at most 168 registers (the instance with
-                                                                  // modified scores needs more and takes an SM alone)
+__global__ void __launch_bounds__(FA_THREADS, MODS & 3 ? 1 : 2)   // two blocks per SM: at most 168 registers (the instances with
+                                                                  // a cap or a bias table need more and take an SM alone)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv activation [tokens, q_stride], box {64, 128}
                             const __grid_constant__ CUtensorMap map_k,   // key pages as rows [pages * kv_heads * page_size, D], box {64, page rows}
                             const __grid_constant__ CUtensorMap map_v,
@@ -358,8 +358,12 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                 const float cap2 = p.mods.softcap * 1.4426950408889634f, in_cap = (MODS & 1) ? p.scale / p.mods.softcap : 0.f;
                 const float* bias_h = (MODS & 2) ? p.mods.dist_bias + (int64_t)head * p.mods.dist_len : nullptr;
                 const unsigned last_dist = (unsigned)(p.mods.dist_len - 1);
-                auto score2 = [&](uint32_t raw, int key) {
+                // A slope: the score of key j takes slope (j - qpos) in base 2.  Within a chunk of 32 keys that is `off` (the chunk's first
+                // key's share, worked out once) plus slope times the key's place in the chunk, a constant of the unrolled loop.
+                const float slope2 = (MODS & 4) ? p.mods.slope[head] * 1.4426950408889634f : 0.f;
+                auto score2 = [&](uint32_t raw, int key, int i, float off) {
                     float x = __uint_as_float(raw);
+                    if (MODS & 4) return fmaf(x, p.scale_log2e, fmaf(slope2, (float)i, off));
                     x = (MODS & 1) ? cap2 * tanh_fast(x * in_cap) : x * p.scale_log2e;
                     // (a key behind the query has a negative distance: as an unsigned number it is clamped like a far one; its score is masked)
                     if (MODS & 2) x = fmaf(bias_h[min((unsigned)(qpos - key), last_dist)], 1.4426950408889634f, x);
@@ -413,9 +417,10 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                         constexpr bool MASK = decltype(mask_tag)::value;
                         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
                         for_each_chunk([&](int ch, const uint32_t* c) {
+                            const float off = (MODS & 4) ? slope2 * (float)(key0 + ch * 32 - qpos) : 0.f;
     #pragma unroll
                             for (int i = 0; i < 32; ++i) {
-                                float x = MODS ? score2(c[i], key0 + ch * 32 + i) : __uint_as_float(c[i]);
+                                float x = MODS ? score2(c[i], key0 + ch * 32 + i, i, off) : __uint_as_float(c[i]);
                                 if (MASK && masked(key0 + ch * 32 + i)) x = -INFINITY;
                                 mx4[i & 3] = fmaxf(mx4[i & 3], x);
                             }
@@ -436,12 +441,13 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                         float xm[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}, sm[4] = {0.f, 0.f, 0.f, 0.f};
                         for_each_chunk([&](int ch, const uint32_t* c) {
                             uint32_t packed[16];
+                            const float off = (MODS & 4) ? fmaf(slope2, (float)(key0 + ch * 32 - qpos), neg_m) : neg_m;     // a slope's chunk takes the reference point in too
                             // P(t-1) must have been read by its product before it is overwritten (normally long done)
                             if (ch == 0 && g > 0 && !__all_sync(0xffffffffu, mbar_wait(&kv_empty[(g - 1) & 1], ((g - 1) >> 1) & 1, abort_p))) ok = false;
     #pragma unroll
                             for (int i = 0; i < 32; i += 2) {
-                                float x0 = MODS ? score2(c[i], key0 + ch * 32 + i) + neg_m : fmaf(__uint_as_float(c[i]), p.scale_log2e, neg_m);
-                                float x1 = MODS ? score2(c[i + 1], key0 + ch * 32 + i + 1) + neg_m : fmaf(__uint_as_float(c[i + 1]), p.scale_log2e, neg_m);
+                                float x0 = MODS & 4 ? score2(c[i], 0, i, off) : MODS ? score2(c[i], key0 + ch * 32 + i, i, 0.f) + neg_m : fmaf(__uint_as_float(c[i]), p.scale_log2e, neg_m);
+                                float x1 = MODS & 4 ? score2(c[i + 1], 0, i + 1, off) : MODS ? score2(c[i + 1], key0 + ch * 32 + i + 1, i + 1, 0.f) + neg_m : fmaf(__uint_as_float(c[i + 1]), p.scale_log2e, neg_m);
                                 if (MASK) {
                                     if (masked(key0 + ch * 32 + i)) x0 = -INFINITY;
                                     if (masked(key0 + ch * 32 + i + 1)) x1 = -INFINITY;
@@ -967,7 +973,7 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
                                         const int* row_q_len, const int* row_ctx_len, int num_rows, int num_tokens, void* out,
                                         int num_heads, int num_kv_heads, int head_dim, int page_size, float scale, int window,
                                         int keep, int min_q_len, int work_rows, int work_tokens, int out_f32, float softcap, const float* sink,
-                                        const float* dist_bias, int dist_len, cudaStream_t stream) {
+                                        const float* dist_bias, int dist_len, const float* slope, cudaStream_t stream) {
     if (num_rows <= 0 || num_tokens <= 0) return 0;
     if (work_rows <= 0 || work_tokens <= 0 || work_rows > num_rows || work_tokens > num_tokens) { work_rows = num_rows; work_tokens = num_tokens; }
     if (head_dim != 64 && head_dim != 128) return MIE_ERR_BAD_ARG;
@@ -987,9 +993,10 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
     p.window = window; p.keep = window && keep > 0 ? keep : 0; p.min_q_len = min_q_len; p.pair = 0;
     p.scale_log2e = scale * 1.4426950408889634f;
     p.scale = scale;
-    p.mods = ScoreMods{softcap, sink, dist_bias, dist_len};
+    p.mods = ScoreMods{softcap, sink, dist_bias, dist_len, slope};
     if (dist_bias && dist_len <= 0) return MIE_ERR_BAD_ARG;
-    const int mods = (softcap > 0.f ? 1 : 0) | (dist_bias ? 2 : 0);
+    const int mods = (softcap > 0.f ? 1 : 0) | (dist_bias ? 2 : 0) | (slope ? 4 : 0);
+    if (mods > 4) return MIE_ERR_BAD_ARG;              // a slope with a cap or a bias: the mma.sync kernel takes those
     p.check_pages = num_pages; p.report = g_range_report;
     CUtensorMap mq, mk, mv;
     const int box_rows = page_size < FA_BN ? page_size : FA_BN;
@@ -999,8 +1006,9 @@ extern "C" int mie_prefill_attention_tc(const void* q, int64_t q_stride, const v
     if ((rc = make_map_2d(&mv, v_cache, cache_rows, (uint64_t)head_dim, (uint64_t)head_dim, box_rows))) return rc;
 #define FA_MODS(DD) (mods == 1 ? launch_fa<DD, 1, false>(mq, mk, mv, p, work_tokens, work_rows, stream)                                  \
                      : mods == 2 ? launch_fa<DD, 2, false>(mq, mk, mv, p, work_tokens, work_rows, stream)                                \
+                     : mods == 4 ? launch_fa<DD, 4, false>(mq, mk, mv, p, work_tokens, work_rows, stream)                                \
                                  : launch_fa<DD, 3, false>(mq, mk, mv, p, work_tokens, work_rows, stream))
-    if (mods && p.keep) return MIE_ERR_BAD_ARG;        // kept keys with a cap or a bias: the mma.sync kernel takes those
+    if (mods && p.keep) return MIE_ERR_BAD_ARG;        // kept keys with a modified score: the mma.sync kernel takes those
     if (mods) return head_dim == 64 ? FA_MODS(64) : FA_MODS(128);
 #undef FA_MODS
     if (p.keep) return head_dim == 64 ? launch_fa<64, 0, true>(mq, mk, mv, p, work_tokens, work_rows, stream)

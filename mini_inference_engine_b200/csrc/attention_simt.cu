@@ -186,11 +186,11 @@ extern "C" int mie_paged_attention(const void* q, int64_t q_stride, const void* 
                                    int num_tokens, void* out, int act_tag, int num_heads, int num_kv_heads,
                                    int head_dim, int page_size, float scale, int window, int keep, int min_q_len,
                                    long long num_pages, int out_f32, float softcap, const float* sink, const float* dist_bias,
-                                   int dist_len, cudaStream_t stream) {
+                                   int dist_len, const float* slope, cudaStream_t stream) {
     if (num_rows <= 0 || num_tokens <= 0) return 0;
     if (head_dim < 16 || head_dim > ATT_MAX_D || head_dim % 16) return MIE_ERR_BAD_ARG;
     if (dist_bias && dist_len <= 0) return MIE_ERR_BAD_ARG;
-    const ScoreMods mods{softcap, sink, dist_bias, dist_len};
+    const ScoreMods mods{softcap, sink, dist_bias, dist_len, slope};
     if (num_kv_heads <= 0 || num_heads % num_kv_heads) return MIE_ERR_BAD_ARG;
     if (page_size < 1 || (page_size & (page_size - 1))) return MIE_ERR_BAD_ARG;
     int page_shift = 0;

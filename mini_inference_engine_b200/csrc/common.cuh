@@ -44,6 +44,7 @@ struct ScoreMods {
     const float* sink;         // not null, [heads]: exp(sink[head]) is one more term of the softmax's denominator (a term without a score or a value of its own)
     const float* dist_bias;    // not null, [heads, dist_len]: the query at position p adds entry min(p - j, dist_len - 1) of its head's row to key j's score
     int dist_len;
+    const float* slope;        // not null, [heads]: slope[head] * (p - j) is taken off key j's score (a bias that grows with the distance, unbounded)
 };
 // tanh as 1 - 2 / (exp(2x) + 1) with the fast exponential and division: absolute error about 1e-7, a handful of instructions
 // where the library's takes thirty and a branch (the kernels on tensor cores, whose products come from bfloat16 operands)
@@ -52,6 +53,7 @@ template <bool FAST = false>
 __device__ __forceinline__ float mod_score(float s, const ScoreMods& m, int head, int num_heads, int dist) {
     if (m.softcap > 0.f) s = m.softcap * (FAST ? tanh_fast(s / m.softcap) : tanhf(s / m.softcap));
     if (m.dist_bias) s += m.dist_bias[head * m.dist_len + min(max(dist, 0), m.dist_len - 1)];
+    if (m.slope) s = fmaf(-m.slope[head], (float)dist, s);
     return s;
 }
 

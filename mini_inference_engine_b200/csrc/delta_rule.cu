@@ -1,7 +1,7 @@
-// The gated delta rule with one decay per head and key channel: a linear-attention mixer whose per-head state
+// The gated delta rule with one decay per head and key channel, or one per head: a linear-attention mixer whose per-head state
 // S [D, Dv] (float32) forgets per key channel, corrects what it holds under the new key, and is read by the query:
 //
-//   S <- diag(g_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t        (in this order)
+//   S <- diag(g_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t        (in this order; g_t may be one number)
 //
 // Three kernels:
 //   prepare    per token: the short causal convolution over time of q, k and v (inputs older than the step's portion come
@@ -38,7 +38,8 @@ __device__ __forceinline__ float conv_at(const T* __restrict__ x, int64_t stride
 }
 
 // proj[t] = [ q: G x D | k: G x D | v: H x Dv | beta logits: H | ... ] (activation type, row stride `stride`);
-// low[t] = [ a: H x D | ... ] float32 (row stride low_stride).  One block per token, one warp per head of q, k or v.
+// low[t] = [ a: H x A | ... ] float32 (row stride low_stride), A decays a head: D, or 1 -- then the beta logits are float32 too and
+// stand behind them, low[t] = [ a: H | beta logits: H | ... ].  One block per token, one warp per head of q, k or v.
 template <typename T>
 __global__ void delta_prepare_kernel(const T* __restrict__ proj, int64_t stride, const float* __restrict__ low, int64_t low_stride,
                                      const float* __restrict__ taps, const float* __restrict__ conv_state,
@@ -46,9 +47,9 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int64_t stride,
                                      const int* __restrict__ state_slots, const float* __restrict__ a_log,
                                      const float* __restrict__ dt_bias, float* __restrict__ qn, float* __restrict__ kn,
                                      float* __restrict__ vn, float* __restrict__ beta, float* __restrict__ decay,
-                                     float* __restrict__ kq, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps) {
+                                     float* __restrict__ kq, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps, int per_head) {
     pdl_enter();
-    const int t = blockIdx.x;
+    const int t = blockIdx.x, A = per_head ? 1 : D;
     const int row = token_row[t];
     const int local = t - row_q_start[row];
     const int C = 2 * G * D + H * Dv;
@@ -89,10 +90,14 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int64_t stride,
         }
     }
     const T* bl = proj + (int64_t)t * stride + C;
-    for (int h = threadIdx.x; h < H; h += blockDim.x) beta[(int64_t)t * H + h] = 1.0f / (1.0f + expf(-to_f32<T>(bl[h])));
-    for (int i = threadIdx.x; i < H * D; i += blockDim.x) {
-        const float rate = expf(a_log[i / D]);
-        decay[(int64_t)t * H * D + i] = expf(-rate * softplus_f(low[(int64_t)t * low_stride + i] + dt_bias[i]));
+    const float* lo = low + (int64_t)t * low_stride;
+    for (int h = threadIdx.x; h < H; h += blockDim.x) {
+        const float z = per_head ? lo[H + h] : to_f32<T>(bl[h]);
+        beta[(int64_t)t * H + h] = 1.0f / (1.0f + expf(-z));
+    }
+    for (int i = threadIdx.x; i < H * A; i += blockDim.x) {
+        const float rate = expf(a_log[i / A]);
+        decay[(int64_t)t * H * A + i] = expf(-rate * softplus_f(lo[i] + dt_bias[i]));
     }
     __syncthreads();                                   // q and k of this token, written above by other warps of the block
     for (int g = warp; g < G; g += nw) {               // k . q per key head: the same for every value column of the recurrence
@@ -141,8 +146,9 @@ __device__ __forceinline__ void cp_async16(float* dst_smem, const float* src) {
 // (asynchronous copies, two batches ahead of the one being computed).  ring[slot] = [k: D | q: D | g: D | v: cols | beta | kq],
 // padded to whole 16-byte pieces.  A lane holds R entries of its column: few, so that a column's sums are spread
 // over many lanes and an SM holds many warps whose chains hide one another's latency.  VEC: D = L * R and D % 4 = 0, so the
-// ring is filled and read 16 bytes at a time and nothing needs a bound check; otherwise everything goes entry by entry.
-template <int R, bool VEC, int LT>
+// ring is filled and read 16 bytes at a time and nothing needs a bound check; otherwise everything goes entry by entry.  ONE: one
+// decay per head -- the ring holds [k | q | v | beta | kq | g], the column's sums are taken before the decay and scaled with it.
+template <int R, bool VEC, int LT, bool ONE>
 __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ vn,
                                   const float* __restrict__ beta, const float* __restrict__ decay, const float* __restrict__ kq,
                                   const int* __restrict__ row_q_start, const int* __restrict__ row_q_len,
@@ -166,7 +172,8 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
         const int i = row_of(r);
         s[r] = (active && i < D) ? sp[i] : 0.f;
     }
-    const int v_at = 3 * D + (cl < cols ? cl : 0);
+    constexpr int SEGS = ONE ? 2 : 3;                          // key-long operands a token: k, q and (a decay per channel) g
+    const int v_at = SEGS * D + (cl < cols ? cl : 0);
     const float v_on = cl < cols ? 1.f : 0.f;
     const int batches = (n + tb - 1) / tb;
     auto issue = [&](int batch) {                              // every thread commits one group per call, also an empty one
@@ -176,7 +183,7 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
             const int64_t tf = t0 + first;
             if constexpr (VEC) {
                 const int q4 = D >> 2;                         // 16-byte pieces of one operand
-                for (int c = threadIdx.x; c < 3 * q4; c += blockDim.x) {
+                for (int c = threadIdx.x; c < SEGS * q4; c += blockDim.x) {
                     const int seg = c / q4, off = (c - seg * q4) * 4;
                     const float* src = seg == 0 ? kn + (tf * G + kh) * D : (seg == 1 ? qn + (tf * G + kh) * D : decay + (tf * H + h) * D);
                     const int64_t step = seg < 2 ? (int64_t)G * D : (int64_t)H * D;
@@ -184,17 +191,18 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
                     for (int tok = 0; tok < count; ++tok) cp_async16(dst + tok * slot_floats, src + off + tok * step);
                 }
             } else {
-                for (int c = threadIdx.x; c < 3 * D; c += blockDim.x) {
+                for (int c = threadIdx.x; c < SEGS * D; c += blockDim.x) {
                     const int seg = c / D, off = c - seg * D;
                     const float* src = seg == 0 ? kn + (tf * G + kh) * D : (seg == 1 ? qn + (tf * G + kh) * D : decay + (tf * H + h) * D);
                     const int64_t step = seg < 2 ? (int64_t)G * D : (int64_t)H * D;
                     for (int tok = 0; tok < count; ++tok) cp_async4(base + tok * slot_floats + c, src + off + tok * step);
                 }
             }
-            for (int c = threadIdx.x; c < cols + 2; c += blockDim.x) {
-                const float* src = c < cols ? vn + (tf * H + h) * Dv + min(j0 + c, Dv - 1) : (c == cols ? beta + tf * H + h : kq + tf * G + kh);
-                const int64_t step = c < cols ? (int64_t)H * Dv : (c == cols ? H : G);
-                for (int tok = 0; tok < count; ++tok) cp_async4(base + tok * slot_floats + 3 * D + c, src + tok * step);
+            for (int c = threadIdx.x; c < cols + (ONE ? 3 : 2); c += blockDim.x) {
+                const float* src = c < cols ? vn + (tf * H + h) * Dv + min(j0 + c, Dv - 1)
+                                            : (c == cols ? beta + tf * H + h : c == cols + 1 ? kq + tf * G + kh : decay + tf * H + h);
+                const int64_t step = c < cols ? (int64_t)H * Dv : (c == cols + 1 ? G : H);
+                for (int tok = 0; tok < count; ++tok) cp_async4(base + tok * slot_floats + SEGS * D + c, src + tok * step);
             }
         }
         cp_async_commit();
@@ -210,14 +218,15 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
 #pragma unroll 4                                              // the next tokens' operands are read while a token's sums travel
         for (int tok = 0; tok < count; ++tok) {
             const float* op = base + tok * slot_floats;
-            float k[R], q[R], g[R];
+            float k[R], q[R], g[ONE ? 1 : R];
+            const float one = ONE ? op[2 * D + cols + 2] : 1.f;
             if constexpr (VEC) {
 #pragma unroll
                 for (int r = 0; r < R; r += 4) {
                     const int i = 4 * (l + L * (r >> 2));
                     *reinterpret_cast<float4*>(k + r) = *reinterpret_cast<const float4*>(op + i);
                     *reinterpret_cast<float4*>(q + r) = *reinterpret_cast<const float4*>(op + D + i);
-                    *reinterpret_cast<float4*>(g + r) = *reinterpret_cast<const float4*>(op + 2 * D + i);
+                    if constexpr (!ONE) *reinterpret_cast<float4*>(g + r) = *reinterpret_cast<const float4*>(op + 2 * D + i);
                 }
             } else {
 #pragma unroll
@@ -226,14 +235,16 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
                     const bool ok = i < D;
                     k[r] = ok ? op[i] : 0.f;
                     q[r] = ok ? op[D + i] : 0.f;
-                    g[r] = ok ? op[2 * D + i] : 0.f;
+                    if constexpr (!ONE) g[r] = ok ? op[2 * D + i] : 0.f;
                 }
             }
             float r1 = 0.f, r2 = 0.f, r1b = 0.f, r2b = 0.f;             // two chains each: half the dependent latency
 #pragma unroll
             for (int r = 0; r < R; r += 2) {
-                s[r] *= g[r];
-                s[r + 1] *= g[r + 1];
+                if constexpr (!ONE) {
+                    s[r] *= g[r];
+                    s[r + 1] *= g[r + 1];
+                }
                 r1 = fmaf(s[r], k[r], r1);
                 r1b = fmaf(s[r + 1], k[r + 1], r1b);
                 r2 = fmaf(s[r], q[r], r2);
@@ -253,10 +264,10 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
                     r2 += __shfl_xor_sync(0xffffffffu, r2, o);
                 }
             }
-            const float u = op[3 * D + cols] * (v_on * op[v_at] - r1);
+            const float u = op[SEGS * D + cols] * (v_on * op[v_at] - one * r1);
 #pragma unroll
-            for (int r = 0; r < R; ++r) s[r] = fmaf(k[r], u, s[r]);
-            if (active && l == 0) out[((int64_t)(t0 + first + tok) * H + h) * Dv + j] = fmaf(u, op[3 * D + cols + 1], r2);
+            for (int r = 0; r < R; ++r) s[r] = fmaf(k[r], u, one * s[r]);
+            if (active && l == 0) out[((int64_t)(t0 + first + tok) * H + h) * Dv + j] = fmaf(u, op[SEGS * D + cols + 1], one * r2);
         }
         __syncthreads();                                       // the slot may be refilled
     }
@@ -269,10 +280,26 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
     }
 }
 
-// out[t, h, :] = o[t, h, :] * rsqrt(mean(o[t, h, :]^2) + eps) * w[:] * sigmoid(gate[t, h, :]); a warp per (token, head).
-// gate: float32 rows of stride gate_stride; w: float32 [Dv] or null.
-template <typename T>
-__global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate, int64_t gate_stride,
+// out[t, h, :] = o[t, h, :] * rsqrt(mean(o[t, h, :]^2) + eps) * w[:] * f(gate[t, h, :]), f the sigmoid or (SILU) z sigmoid(z); a warp per
+// (token, head), four consecutive entries a lane where rows are whole 16-byte pieces (VEC), the head's entries in registers between
+// the statistic and the output.  gate: rows of stride gate_stride; w: float32 [Dv] or null.
+__device__ __forceinline__ float4 head_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 head_load4(const bf16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void head_store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void head_store4(bf16* p, const float4& v) {
+    uint2 u;
+    *reinterpret_cast<__nv_bfloat162*>(&u.x) = __floats2bfloat162_rn(v.x, v.y);
+    *reinterpret_cast<__nv_bfloat162*>(&u.y) = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = u;
+}
+template <bool SILU> __device__ __forceinline__ float gate_of(float z) { return (SILU ? z : 1.0f) / (1.0f + expf(-z)); }
+
+template <typename T, typename TG, bool SILU, bool VEC>
+__global__ void head_norm_gate_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int64_t gate_stride,
                                       const float* __restrict__ w, T* __restrict__ out, int num_tokens, int H, int Dv, float eps) {
     pdl_enter();
     const int lane = threadIdx.x & 31;
@@ -281,14 +308,35 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
     const int64_t t = item / H;
     const int h = (int)(item - t * H);
     const float* src = o + item * Dv;
+    const TG* g = gate ? gate + t * gate_stride + (int64_t)h * Dv : nullptr;
+    if constexpr (VEC) {
+        float4 v[2];                                               // heads of up to 256 entries
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int i = 4 * lane + 128 * k;
+            v[k] = i < Dv ? head_load4(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+        }
+        const float s = 1.0f / sqrtf(warp_sum(ss) / (float)Dv + eps);
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int i = 4 * lane + 128 * k;
+            if (i >= Dv) continue;
+            float4 y = make_float4(v[k].x * s, v[k].y * s, v[k].z * s, v[k].w * s);
+            if (w) { const float4 u = head_load4(w + i); y.x *= u.x; y.y *= u.y; y.z *= u.z; y.w *= u.w; }
+            if (g) { const float4 u = head_load4(g + i); y.x *= gate_of<SILU>(u.x); y.y *= gate_of<SILU>(u.y); y.z *= gate_of<SILU>(u.z); y.w *= gate_of<SILU>(u.w); }
+            head_store4(out + item * Dv + i, y);
+        }
+        return;
+    }
     float ss = 0.f;
     for (int i = lane; i < Dv; i += 32) { const float v = src[i]; ss += v * v; }
     const float s = 1.0f / sqrtf(warp_sum(ss) / (float)Dv + eps);
-    const float* g = gate ? gate + t * gate_stride + (int64_t)h * Dv : nullptr;
     for (int i = lane; i < Dv; i += 32) {
         float v = src[i] * s;
         if (w) v *= w[i];
-        if (g) v /= 1.0f + expf(-g[i]);
+        if (g) v *= gate_of<SILU>(to_f32<TG>(g[i]));
         out[item * Dv + i] = from_f32<T>(v);
     }
 }
@@ -296,7 +344,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
 extern "C" int mie_delta_prepare(const void* proj, int tag, long long stride, const float* low, long long low_stride, const float* taps,
                                  const float* conv_state, const int* token_row, const int* row_q_start, const int* state_slots,
                                  const float* a_log, const float* dt_bias, float* qn, float* kn, float* vn, float* beta, float* decay,
-                                 float* kq, int num_tokens, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps,
+                                 float* kq, int num_tokens, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps, int per_head,
                                  cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || K < 1) return MIE_ERR_BAD_ARG;
@@ -305,11 +353,11 @@ extern "C" int mie_delta_prepare(const void* proj, int tag, long long stride, co
     if (tag == MIE_F32)
         return launch_kernel(delta_prepare_kernel<float>, dim3(num_tokens), dim3(threads), 0, stream, (const float*)proj, (int64_t)stride,
                              low, (int64_t)low_stride, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias, qn, kn, vn,
-                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps);
+                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps, per_head);
     else if (tag == MIE_BF16)
         return launch_kernel(delta_prepare_kernel<bf16>, dim3(num_tokens), dim3(threads), 0, stream, (const bf16*)proj, (int64_t)stride,
                              low, (int64_t)low_stride, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias, qn, kn, vn,
-                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps);
+                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps, per_head);
     return MIE_ERR_BAD_ARG;
 }
 
@@ -328,7 +376,7 @@ extern "C" int mie_conv_state_update(const void* x, int tag, long long stride, c
     return MIE_ERR_BAD_ARG;
 }
 
-template <int R>
+template <int R, bool ONE>
 static int launch_scan(const float* qn, const float* kn, const float* vn, const float* beta, const float* decay, const float* kq,
                        const int* row_q_start, const int* row_q_len, const int* state_slots, float* state, float* out, int num_rows,
                        int H, int G, int D, int Dv, cudaStream_t stream) {
@@ -340,16 +388,16 @@ static int launch_scan(const float* qn, const float* kn, const float* vn, const 
     const int threads = (cols * L + 31) / 32 * 32;
     const dim3 grid(num_rows, H, (Dv + cols - 1) / cols);
     // tokens a batch of the ring: eight where three such batches stay within 48 KB, fewer for long keys
-    const int slot_floats = (3 * D + cols + 2 + 3) / 4 * 4;
+    const int slot_floats = ((ONE ? 2 : 3) * D + cols + (ONE ? 3 : 2) + 3) / 4 * 4;
     const size_t slot_bytes = (size_t)slot_floats * sizeof(float);
     int tb = (int)(48 * 1024 / (DELTA_BATCHES * slot_bytes));
     if (tb > 8) tb = 8;
     if (tb < 1) tb = 1;
     const size_t smem = (size_t)DELTA_BATCHES * tb * slot_bytes;
     const bool vec = D == L * R && D % 4 == 0 &&
-                     ((reinterpret_cast<uintptr_t>(qn) | reinterpret_cast<uintptr_t>(kn) | reinterpret_cast<uintptr_t>(decay)) & 15) == 0;
+                     ((reinterpret_cast<uintptr_t>(qn) | reinterpret_cast<uintptr_t>(kn) | (ONE ? 0 : reinterpret_cast<uintptr_t>(decay))) & 15) == 0;
     // the vectorised kernel with the lanes a column as a constant for the common key sizes (64 and 128: 16 lanes), else at run time
-    auto kernel = !vec ? delta_scan_kernel<R, false, 0> : (L == 16 ? delta_scan_kernel<R, true, 16> : delta_scan_kernel<R, true, 0>);
+    auto kernel = !vec ? delta_scan_kernel<R, false, 0, ONE> : (L == 16 ? delta_scan_kernel<R, true, 16, ONE> : delta_scan_kernel<R, true, 0, ONE>);
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
@@ -360,28 +408,39 @@ static int launch_scan(const float* qn, const float* kn, const float* vn, const 
 
 extern "C" int mie_delta_scan(const float* qn, const float* kn, const float* vn, const float* beta, const float* decay, const float* kq,
                               const int* row_q_start, const int* row_q_len, const int* state_slots, float* state, float* out,
-                              int num_rows, int H, int G, int D, int Dv, cudaStream_t stream) {
+                              int num_rows, int H, int G, int D, int Dv, int A, cudaStream_t stream) {
     if (num_rows <= 0) return 0;
-    if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0) return MIE_ERR_BAD_ARG;
+    if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || (A != 1 && A != D)) return MIE_ERR_BAD_ARG;
     // entries of a column a lane: the fewest for which sixteen lanes hold a column (thirty-two for the longest keys)
-    if (D <= 64) return launch_scan<4>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, stream);
-    if (D <= 128) return launch_scan<8>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, stream);
-    if (D <= DELTA_MAX_KEY) return launch_scan<16>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, stream);
+#define SCAN(R) (A == 1 ? launch_scan<R, true>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, stream)  \
+                        : launch_scan<R, false>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, stream))
+    if (D <= 64) return SCAN(4);
+    if (D <= 128) return SCAN(8);
+    if (D <= DELTA_MAX_KEY) return SCAN(16);
+#undef SCAN
     return MIE_ERR_TOO_LARGE;
 }
 
-extern "C" int mie_head_norm_gate(const float* o, const float* gate, long long gate_stride, const float* w, void* out, int tag,
-                                  int num_tokens, int H, int Dv, float eps, cudaStream_t stream) {
+template <typename T, typename TG, bool SILU>
+static int launch_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, const float* w, void* out, int num_tokens, int H,
+                                 int Dv, float eps, cudaStream_t stream) {
+    const int warps = 4;
+    const int blocks = (int)(((int64_t)num_tokens * H + warps - 1) / warps);
+    const auto whole = [](const void* p, uintptr_t bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
+    const bool vec = Dv % 4 == 0 && Dv <= 256 && gate_stride % 4 == 0 && whole(o, 16) && whole(w, 16) && whole(gate, 4 * sizeof(TG)) && whole(out, 4 * sizeof(T));
+    return launch_kernel(vec ? head_norm_gate_kernel<T, TG, SILU, true> : head_norm_gate_kernel<T, TG, SILU, false>, dim3(blocks), dim3(warps * 32), 0,
+                         stream, o, (const TG*)gate, gate_stride, w, (T*)out, num_tokens, H, Dv, eps);
+}
+
+// gate_tag: the gate's type (float32, or the output's); silu: the gate is z sigmoid(z), else sigmoid(z).
+extern "C" int mie_head_norm_gate(const float* o, const void* gate, int gate_tag, long long gate_stride, const float* w, void* out, int tag,
+                                  int num_tokens, int H, int Dv, float eps, int silu, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (H <= 0 || Dv <= 0) return MIE_ERR_BAD_ARG;
-    const int warps = 4;
-    const int64_t items = (int64_t)num_tokens * H;
-    const int blocks = (int)((items + warps - 1) / warps);
-    if (tag == MIE_F32)
-        return launch_kernel(head_norm_gate_kernel<float>, dim3(blocks), dim3(warps * 32), 0, stream, o, gate, (int64_t)gate_stride, w,
-                             (float*)out, num_tokens, H, Dv, eps);
-    else if (tag == MIE_BF16)
-        return launch_kernel(head_norm_gate_kernel<bf16>, dim3(blocks), dim3(warps * 32), 0, stream, o, gate, (int64_t)gate_stride, w,
-                             (bf16*)out, num_tokens, H, Dv, eps);
+#define HNG(T, TG) (silu ? launch_head_norm_gate<T, TG, true>(o, gate, gate_stride, w, out, num_tokens, H, Dv, eps, stream)  \
+                         : launch_head_norm_gate<T, TG, false>(o, gate, gate_stride, w, out, num_tokens, H, Dv, eps, stream))
+    if (tag == MIE_F32) return gate_tag == MIE_F32 ? HNG(float, float) : MIE_ERR_BAD_ARG;
+    if (tag == MIE_BF16) return gate_tag == MIE_F32 ? HNG(bf16, float) : HNG(bf16, bf16);
+#undef HNG
     return MIE_ERR_BAD_ARG;
 }

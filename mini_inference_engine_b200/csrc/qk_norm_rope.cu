@@ -14,6 +14,7 @@
 // are null (heads of unit root mean square; a statistic over whole pairs is the same before and after the rotation, which
 // changes no pair's length, so this also serves designs that norm the rotated heads);
 // `v_freq` (Dv/2 float32, or null) -- v is rotated too, over all its Dv entries in the same pairing, before it is stored;
+// `v_cache` null -- there are no values of their own (the keys serve as values): rows hold q and k only, and only k is stored;
 // `interleaved` -- the rotation pairs entry 2i with 2i + 1 instead of i with i + rot/2 (the same angle position * freq[i]);
 // `temp_coef`, `temp_every` -- the query of position p is also multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
 // (a temperature that grows with the position; temp_every <= 0: none).
@@ -113,6 +114,7 @@ __global__ void qk_norm_rope_kernel(const T* __restrict__ qkv, int64_t qkv_strid
         const float s_g = head_norm ? head_scale(k, g, lane) : sk;
         for (int d = lane; d < DP; d += 32) {
             k_cache[row + d] = from_f32<T>(d < D ? entry(k, kw, s_g, g, d) * k_scale : 0.f);
+            if (!v_cache) continue;
             if (!v_freq || d >= Dv) {
                 v_cache[row + d] = d < Dv ? v[g * Dv + d] : from_f32<T>(0.f);
                 continue;
@@ -188,7 +190,7 @@ __global__ void qk_norm_rope_bf16x8_kernel(const QkVec p) {
     const int slot = p.write_cache ? p.slots[t] : 0;
     const bool stores = p.write_cache && range_slot(slot, p.num_pages, p.page_size) == MIE_RANGE_OK;
     if (p.write_cache && !stores && threadIdx.x == 0) range_report(p.report, MIE_RANGE_SLOT, MIE_K_QK_NORM_ROPE, t, slot);
-    const int heads = p.H + (stores ? 2 * p.G : 0), qk = p.H + p.G;
+    const int heads = p.H + (stores ? (p.v_cache ? 2 : 1) * p.G : 0), qk = p.H + p.G;
     // a head's entries lie side by side: q and k heads are D wide, v heads Dv
     auto load = [&](int hh) {
         const int width = hh < qk ? p.D : p.Dv;
@@ -270,7 +272,7 @@ __global__ void qk_norm_rope_bf16x8_kernel(const QkVec p) {
 
 template <int LANES>
 static int launch_qk_vec(const QkVec& p, int num_tokens, cudaStream_t stream) {
-    const int pieces = (p.H + 2 * p.G) * LANES;
+    const int pieces = (p.H + (p.v_cache ? 2 : 1) * p.G) * LANES;
     int threads = 64;
     while (threads < 256 && threads < pieces) threads <<= 1;
     return launch_kernel(qk_norm_rope_bf16x8_kernel<LANES>, dim3(num_tokens), dim3(threads),

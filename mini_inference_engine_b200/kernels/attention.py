@@ -63,7 +63,7 @@ def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, wi
     where ``rotates_in_decode`` holds.  ``window``: None or 0 all earlier keys, w > 0 the last w positions, w < 0 the
     keys of the query's own block of -w positions.  ``keep``: beside a window or block, the first ``keep`` keys of the
     sequence stay in sight.  ``q_stride``: elements between the token rows of ``qkv`` (by
-    default rows of a fused q|k|v projection).  ``mods`` (``ops.ScoreMods``): a cap on the scores, a bias by distance, a sink in
+    default rows of a fused q|k|v projection).  ``mods`` (``ops.ScoreMods``): a cap on the scores, a bias or a slope by distance, a sink in
     the softmax; every kernel applies them (the tcgen05 kernel for portions in an instance of its own)."""
     if q_stride is None:
         q_stride = (num_heads + 2 * num_kv_heads) * head_dim
@@ -98,9 +98,9 @@ def attention(qkv, ctx, cache, out, num_heads, num_kv_heads, head_dim, scale, wi
                              max_ctx=reach, mods=mods, keep=keep)
     if has_prefill:
         # tcgen05 (S and O in tensor memory) for the head sizes it is written for, mma.sync otherwise
-        # (kept keys with a cap or a bias by distance: mma.sync, the tcgen05 kernel has no instance for them)
+        # (combinations of kept keys and score modifiers that the tcgen05 kernel has no instance for: mma.sync)
         tc = (head_dim in (64, 128) and cache.page_size >= 8 and q_stride % 8 == 0 and _prefill_backend == "tcgen05"
-              and not (keep and mods is not None and (mods.softcap > 0 or mods.dist_bias is not None)))
+              and (mods is None or mods.tcgen05_takes(keep)))
         fn = ops.prefill_attention_tc if tc else ops.prefill_attention
         # the rows that are portions, and their tokens: the launch is laid out for those, not for every decoding row
         work = None if kinds is None else (kinds[1], kinds[2])

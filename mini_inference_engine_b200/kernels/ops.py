@@ -78,7 +78,8 @@ _RANGE_CODES = {1: "token id outside the vocabulary (or the fed-back tokens)", 2
                 4: "block-table entry outside the page pool", 5: "row index outside the batch"}
 _RANGE_KERNELS = {1: "embedding", 2: "rope_cache", 3: "norm", 4: "attention_simt", 5: "attention_decode",
                   6: "attention_prefill", 7: "attention_prefill_tc", 8: "gemm_tcgen05 (q|k|v with rotation)",
-                  9: "norm_group", 10: "qk_norm_rope", 11: "hyper_norm", 12: "latent_kv"}
+                  9: "norm_group", 10: "qk_norm_rope", 11: "hyper_norm", 12: "latent_kv",
+                  13: "sandwich_norm"}
 _range_report: torch.Tensor | None = None
 _range_told: set = set()
 
@@ -291,6 +292,31 @@ def add_layernorm(res: torch.Tensor, weight: torch.Tensor, eps: float, out: torc
     return out
 
 
+def sandwich_norm(res: torch.Tensor, eps: float, *, weight=None, out=None, deltas=(), coefs=(), delta_weight=None, extra=None, shift=None,
+                  rows=None) -> torch.Tensor:
+    """res <- res + n(sum_k coefs[k] deltas[k]) * delta_weight + extra + shift in place (n(y) = y / sqrt(mean(y^2) + eps) per row; up to
+    two addends, float32 or bfloat16; ``extra`` float32 of the stream's shape, ``shift`` float32 [n]; everything optional), then
+    out = n(res) * weight where ``out`` is given.  With ``rows`` output row b comes from row rows[b] and the stream is left as it is."""
+    T, n = res.shape
+    _need(res.dtype == torch.float32 and res.is_contiguous(), "the stream must be contiguous float32")
+    for w, name in ((weight, "norm weight"), (delta_weight, "weight of the addends' norm"), (shift, "shift")):
+        if w is not None:
+            _f32(w, name, n)
+    if extra is not None:
+        _f32(extra, "extra", T * n)
+    n_out = T
+    if rows is not None:
+        _i32(rows, "rows")
+        n_out = rows.numel()
+    if out is not None:
+        _need(weight is not None and out.is_contiguous() and tuple(out.shape) == (n_out, n), "norm output shape, and a weight for it")
+    _need(not deltas or delta_weight is not None, "addends are normed with a weight")
+    _check(load("sandwich_norm").mie_sandwich_norm(_ptr(res), *_delta_args(deltas, coefs, res.shape), _ptr(delta_weight), _ptr(extra), _ptr(shift),
+                                                   _ptr(weight), _ptr(out), tag(out) if out is not None else 0, _ptr(rows), n_out, n,
+                                                   ctypes.c_float(eps), T, _stream()), "sandwich_norm")
+    return out
+
+
 def stream_join(res: torch.Tensor, extra: torch.Tensor, out: torch.Tensor, *, deltas=(), coefs=(), res_coef: float = 1.0) -> torch.Tensor:
     """out[t] = [res_coef res[t] + sum_k coefs[k] deltas[k][t] | extra[t]] in out's type (the stream is not written)."""
     T, n = res.shape
@@ -346,10 +372,11 @@ class ScoreMods:
     """What an attention kernel does to a score between the scaled product and the softmax.  ``softcap`` c > 0: s <- c tanh(s / c).
     ``dist_bias`` float32 [heads, L]: the query at position p adds entry min(p - j, L - 1) of its head's row to the score of key j
     (after the cap).
+    ``slope`` float32 [heads]: slope[head] (p - j) is taken off the score.
     ``sink`` float32 [heads]: exp(sink[head]) is one more term of the softmax's denominator: a key that nothing scores and that carries no value."""
 
-    def __init__(self, softcap: float = 0.0, sink=None, dist_bias=None):
-        self.softcap, self.sink, self.dist_bias = float(softcap or 0.0), sink, dist_bias
+    def __init__(self, softcap: float = 0.0, sink=None, dist_bias=None, slope=None):
+        self.softcap, self.sink, self.dist_bias, self.slope = float(softcap or 0.0), sink, dist_bias, slope
 
     def args(self, num_heads: int):
         if self.sink is not None:
@@ -357,8 +384,16 @@ class ScoreMods:
         if self.dist_bias is not None:
             _need(self.dist_bias.dtype == torch.float32 and self.dist_bias.is_contiguous() and self.dist_bias.dim() == 2
                   and self.dist_bias.shape[0] == num_heads and self.dist_bias.shape[1] >= 1, "distance bias must be float32 [heads, L]")
+        if self.slope is not None:
+            _need(self.slope.dtype == torch.float32 and self.slope.is_contiguous() and self.slope.numel() == num_heads, "one float32 slope per head")
         return (ctypes.c_float(self.softcap), _ptr(self.sink), _ptr(self.dist_bias),
-                int(self.dist_bias.shape[1]) if self.dist_bias is not None else 0)
+                int(self.dist_bias.shape[1]) if self.dist_bias is not None else 0, _ptr(self.slope))
+
+    def tcgen05_takes(self, keep: int) -> bool:
+        """Whether the tcgen05 kernel for portions has an instance for these modifiers: any of cap and bias, or a slope alone; beside
+        kept keys none of the three."""
+        modified = self.softcap > 0 or self.dist_bias is not None
+        return not (keep and (modified or self.slope is not None)) and not (modified and self.slope is not None)
 
 
 _NO_MODS = ScoreMods()
@@ -426,8 +461,7 @@ def prefill_attention_tc(q: torch.Tensor, q_stride: int, k_cache, v_cache, block
                          head_dim: int, page_size: int, scale: float, window: int | None = None,
                          min_q_len: int = 2, work=None, mods: ScoreMods | None = None, keep: int = 0) -> torch.Tensor:
     """Causal attention of prompt portions on tcgen05 (S and O in tensor memory, operands by TMA);
-    head_dim 64 or 128.  ``work``: as for ``prefill_attention``.  Kept keys (``keep``) go with a plain score or a sink, not with a cap or
-    a bias."""
+    head_dim 64 or 128.  ``work``: as for ``prefill_attention``.  Which modifiers go together: ``ScoreMods.tcgen05_takes``."""
     _need(q.dtype == torch.bfloat16 == k_cache.dtype == v_cache.dtype and out.dtype in (torch.bfloat16, torch.float32),
           "prefill attention is bfloat16 (its output bfloat16 or float32)")
     _need(head_dim in (64, 128), f"head_dim {head_dim}: the tcgen05 prefill kernel takes 64 and 128")
@@ -781,14 +815,16 @@ def qk_norm_rope(qkv: torch.Tensor, positions, slots, freq: torch.Tensor, q_out:
     over their first ``rot`` dims (pairs (i, i + rot/2), or (2i, 2i + 1) with ``interleaved``), q scaled per head and, with
     ``pos_temp`` = (coef, every), by 1 + coef ln(floor((position + 1) / every) + 1); q written to ``q_out`` [T, H, DP] and k, v
     to their cache slots (pages [page, G, page_size, DP], tails zero).  ``v_freq`` (vdim / 2): v is rotated too, over all its
-    dims, in the same pairing."""
+    dims, in the same pairing.  ``v_cache`` None: the keys serve as values; the rows hold q and k and only k is stored."""
     T = qkv.shape[0]
     DP = q_out.shape[-1]
+    _need(v_cache is not None or v_freq is None, "values that rotate need pages of their own")
     _need(qkv.dim() == 2 and qkv.stride(1) == 1
-          and qkv.shape[1] >= (num_heads * dim + (num_kv_heads * (dim + vdim) if write_cache else 0)),
+          and qkv.shape[1] >= (num_heads * dim + (num_kv_heads * (dim + (vdim if v_cache is not None else 0)) if write_cache else 0)),
           "qkv rows must hold q, k and v (q alone when the cache is not written)")
     _need(q_out.is_contiguous() and q_out.shape == (T, num_heads, DP) and q_out.dtype == qkv.dtype, "q_out must be [T, H, DP]")
-    _need(k_cache.dtype == qkv.dtype == v_cache.dtype and k_cache.shape[-1] == DP and k_cache.is_contiguous(), "cache type and width")
+    _need(k_cache.dtype == qkv.dtype and (v_cache is None or v_cache.dtype == qkv.dtype) and k_cache.shape[-1] == DP and k_cache.is_contiguous(),
+          "cache type and width")
     _need(freq.dtype == torch.float32 and freq.numel() * 2 == rot and freq.is_contiguous(), "one float32 frequency per rotated pair")
     _i32(positions, "positions")
     _i32(slots, "slots")
@@ -1147,23 +1183,27 @@ def diff_combine(maps: torch.Tensor, gate, out: torch.Tensor, *, num_heads: int,
 # --------------------------------------------------------------------------- gated delta rule
 
 def delta_prepare(proj: torch.Tensor, low: torch.Tensor, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias,
-                  qn, kn, vn, beta, decay, kq, *, num_heads: int, num_kv_heads: int, dim: int, vdim: int, unit_eps: float) -> None:
+                  qn, kn, vn, beta, decay, kq, *, num_heads: int, num_kv_heads: int, dim: int, vdim: int, unit_eps: float,
+                  per_head: bool = False) -> None:
     """From rows [q: G x dim | k: G x dim | v: H x vdim | beta logits: H | ...] of the input projection and float32 rows
     [a: H x dim | ...] of the low-rank one: convolution over time + silu of q, k, v (float32 taps [channels, K], older inputs
     from ``conv_state`` [slots, K - 1, channels]), q and k unit vectors per head (q times dim^-1/2), beta = sigmoid,
-    decay = exp(-exp(a_log[h]) softplus(a + dt_bias)), kq = k . q per key head.  All outputs float32."""
+    decay = exp(-exp(a_log[h]) softplus(a + dt_bias)), kq = k . q per key head.  All outputs float32.  ``per_head``: one decay per head (``decay`` [T, H]);
+    the float32 rows are [a: H | beta logits: H | ...] and the projection's hold q, k and v only."""
     T = proj.shape[0]
     H, G, D, Dv = num_heads, num_kv_heads, dim, vdim
     C = 2 * G * D + H * Dv
     K = taps.shape[1]
-    _need(proj.dim() == 2 and proj.stride(1) == 1 and proj.shape[1] >= C + H, "projection rows must hold q, k, v and beta")
-    _need(low.dtype == torch.float32 and low.stride(1) == 1 and low.shape[0] == T and low.shape[1] >= H * D, "low-rank rows must be float32")
+    A = 1 if per_head else D                                         # decays a head
+    _need(proj.dim() == 2 and proj.stride(1) == 1 and proj.shape[1] >= C + (0 if per_head else H), "projection rows must hold q, k, v and beta")
+    _need(low.dtype == torch.float32 and low.stride(1) == 1 and low.shape[0] == T and low.shape[1] >= (2 * H if per_head else H * D),
+          "the decays' rows must be float32")
     _f32(taps, "taps", C * K)
     _need(conv_state.dtype == torch.float32 and conv_state.is_contiguous() and tuple(conv_state.shape[1:]) == (max(K - 1, 0), C),
           "convolution state must be float32 [slots, K - 1, channels]")
     _f32(a_log, "A_log", H)
-    _f32(dt_bias, "dt_bias", H * D)
-    for t, n in ((qn, G * D), (kn, G * D), (vn, H * Dv), (beta, H), (decay, H * D), (kq, G)):
+    _f32(dt_bias, "dt_bias", H * A)
+    for t, n in ((qn, G * D), (kn, G * D), (vn, H * Dv), (beta, H), (decay, H * A), (kq, G)):
         _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n), "outputs must be float32 [T, n]")
     for t, n in ((token_row, "token_row"), (row_q_start, "row_q_start"), (state_slots, "state_slots")):
         _i32(t, n)
@@ -1171,7 +1211,7 @@ def delta_prepare(proj: torch.Tensor, low: torch.Tensor, taps, conv_state, token
     _check(lib.mie_delta_prepare(_ptr(proj), tag(proj), ctypes.c_longlong(proj.stride(0)), _ptr(low), ctypes.c_longlong(low.stride(0)),
                                  _ptr(taps), _ptr(conv_state), _ptr(token_row), _ptr(row_q_start), _ptr(state_slots), _ptr(a_log),
                                  _ptr(dt_bias), _ptr(qn), _ptr(kn), _ptr(vn), _ptr(beta), _ptr(decay), _ptr(kq), T, H, G, D, Dv, K,
-                                 ctypes.c_float(D ** -0.5), ctypes.c_float(unit_eps), _stream()), "delta_prepare")
+                                 ctypes.c_float(D ** -0.5), ctypes.c_float(unit_eps), int(per_head), _stream()), "delta_prepare")
 
 
 def conv_state_update(x: torch.Tensor, row_q_start, row_q_len, state_slots, conv_state) -> None:
@@ -1190,33 +1230,36 @@ def conv_state_update(x: torch.Tensor, row_q_start, row_q_len, state_slots, conv
 def delta_scan(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, *, num_heads: int, num_kv_heads: int,
                dim: int, vdim: int) -> torch.Tensor:
     """S <- decay S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q for every new token of every row, from and to
-    ``state`` [slots, H, vdim, dim] float32.  ``out`` [T, H * vdim] float32."""
+    ``state`` [slots, H, vdim, dim] float32.  ``decay`` [T, H * dim], or [T, H]: one per head.  ``out`` [T, H * vdim] float32."""
     T = qn.shape[0]
     H, G, D, Dv = num_heads, num_kv_heads, dim, vdim
+    A = decay.shape[1] // H
+    _need(A in (1, D), "one decay per head, or one per head and key channel")
     _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, Dv, D), "state must be float32 [slots, H, vdim, dim]")
-    for t, n in ((qn, G * D), (kn, G * D), (vn, H * Dv), (beta, H), (decay, H * D), (kq, G), (out, H * Dv)):
+    for t, n in ((qn, G * D), (kn, G * D), (vn, H * Dv), (beta, H), (decay, H * A), (kq, G), (out, H * Dv)):
         _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n), "operands must be float32 [T, n]")
     for t, n in ((row_q_start, "row_q_start"), (row_q_len, "row_q_len"), (state_slots, "state_slots")):
         _i32(t, n)
     lib = load("delta_rule")
     _check(lib.mie_delta_scan(_ptr(qn), _ptr(kn), _ptr(vn), _ptr(beta), _ptr(decay), _ptr(kq), _ptr(row_q_start), _ptr(row_q_len),
-                              _ptr(state_slots), _ptr(state), _ptr(out), row_q_len.numel(), H, G, D, Dv, _stream()), "delta_scan")
+                              _ptr(state_slots), _ptr(state), _ptr(out), row_q_len.numel(), H, G, D, Dv, A, _stream()), "delta_scan")
     return out
 
 
-def head_norm_gate(o: torch.Tensor, gate, weight, out: torch.Tensor, num_heads: int, vdim: int, eps: float) -> torch.Tensor:
-    """out[t, h] = o[t, h] / rms(o[t, h]) * weight * sigmoid(gate[t, h]) per head of ``vdim`` entries; ``gate`` float32
-    [T, H * vdim], may be a column slice; ``weight`` float32 [vdim]; either may be None."""
+def head_norm_gate(o: torch.Tensor, gate, weight, out: torch.Tensor, num_heads: int, vdim: int, eps: float, silu: bool = False) -> torch.Tensor:
+    """out[t, h] = o[t, h] / rms(o[t, h]) * weight * sigmoid(gate[t, h]) per head of ``vdim`` entries (``silu``: times the gate besides);
+    ``gate`` [T, H * vdim], float32 or of the output's type, may be a column slice; ``weight`` float32 [vdim]; either may be None."""
     T = o.shape[0]
     _need(o.dtype == torch.float32 and o.is_contiguous() and o.shape == (T, num_heads * vdim), "o must be float32 [T, H * vdim]")
     if gate is not None:
-        _need(gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape == o.shape, "gate must be float32 [T, H * vdim]")
+        _need(gate.dtype in (torch.float32, out.dtype) and gate.stride(1) == 1 and gate.shape == o.shape, "gate must be [T, H * vdim], float32 or of the output's type")
     if weight is not None:
         _f32(weight, "head norm weight", vdim)
     _need(out.is_contiguous() and out.shape == o.shape, "out must be contiguous [T, H * vdim]")
     lib = load("delta_rule")
-    _check(lib.mie_head_norm_gate(_ptr(o), _ptr(gate), ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _ptr(weight),
-                                  _ptr(out), tag(out), T, num_heads, vdim, ctypes.c_float(eps), _stream()), "head_norm_gate")
+    _check(lib.mie_head_norm_gate(_ptr(o), _ptr(gate), tag(gate) if gate is not None else 0,
+                                  ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _ptr(weight), _ptr(out), tag(out), T, num_heads,
+                                  vdim, ctypes.c_float(eps), int(silu), _stream()), "head_norm_gate")
     return out
 
 

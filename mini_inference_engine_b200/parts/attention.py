@@ -113,7 +113,10 @@ class GatedAttention(Mixer):
       row n for n < rows / 2, else min(rows - 1, rows/2 + floor(ln(n / (rows/2)) / ln(far / (rows/2)) (rows - rows/2)));
       ``rows`` None: the table's rows come from the checkpoint's tensor (a random model gets 32);
     * ``sink``: a learned number per head ('sink') whose exponential is one more term of the softmax's denominator (nothing is scored for it,
-      nothing read); "one": the term is 1 (a score of 0) for every head and nothing is learned.
+      nothing read); "one": the term is 1 (a score of 0) for every head and nothing is learned;
+    * ``slopes`` (one number a head): slope x (p - j) is taken off the score of the key at j for the query at p;
+    * ``keys_as_values``: there is no value projection, the value at a position is its key as projected (so nothing may norm or turn the
+      keys, and ``vdim`` is ``dim``); a position is stored once and the pages serve as both.
 
     q, k, v and the gate are one product; norm, rotation, temperature and the cache write one kernel; attention
     itself is the framework's paged kernels (decode and portions); the gate one more."""
@@ -122,7 +125,7 @@ class GatedAttention(Mixer):
                  rot_dims: int, rot_base: float, eps: float, rot_scaling: dict | None = None, qk_norm: bool = True,
                  head_temp: bool = True, gate: bool = True, chunk: int | None = None, window: int | None = None,
                  bias: bool = False, rot_pairing: str = "half", q_temp=None, softcap: float = 0.0, rel_bias=None,
-                 sink=False, rotate_values: bool = False, keep_first: int = 0):
+                 sink=False, rotate_values: bool = False, keep_first: int = 0, slopes=None, keys_as_values: bool = False):
         if rot_pairing not in ("half", "interleaved"):
             raise ValueError(f"rot_pairing {rot_pairing!r}; half or interleaved")
         if qk_norm not in (True, False, "head", "projection", "unit"):
@@ -135,6 +138,11 @@ class GatedAttention(Mixer):
             raise ValueError(f"values of {vdim} entries do not rotate in pairs")
         if keep_first < 0:
             raise ValueError("keep_first must not be negative")
+        if slopes is not None and len(slopes) != num_heads:
+            raise ValueError(f"{len(slopes)} slopes for {num_heads} heads")
+        if keys_as_values and (rot_dims or qk_norm or rotate_values or bias or vdim != dim):
+            raise ValueError("keys that serve as values are neither normed, turned nor biased, and have the values' size")
+        self.slopes, self.keys_as_values = tuple(float(s) for s in slopes) if slopes is not None else None, bool(keys_as_values)
         if rel_bias is not None and rel_bias[0] is not None and (int(rel_bias[0]) < 2 or float(rel_bias[1]) <= int(rel_bias[0]) // 2):
             raise ValueError(f"rel_bias {rel_bias!r}: two rows or more, and a far distance beyond half of them")
         self.bias, self.rot_pairing, self.softcap, self.sink = bool(bias), rot_pairing, float(softcap or 0.0), sink
@@ -152,12 +160,16 @@ class GatedAttention(Mixer):
         self.scale, self.eps = float(scale), eps
         self.rot_dims, self.rot_base, self.rot_scaling = rot_dims, rot_base, rot_scaling
         self.qk_norm, self.head_temp, self.gate, self.chunk, self.window = qk_norm, head_temp, gate, chunk, window
-        self.need = KVNeed(num_kv_heads, self.padded, window, chunk, self.keep_first)
+        self.need = KVNeed(num_kv_heads, self.padded, window, chunk, self.keep_first, self.keys_as_values)
+        self.in_names = ("q", "k") if keys_as_values else ("q", "k", "v")
+        self.gate_at = (num_heads + num_kv_heads) * dim + (0 if keys_as_values else num_kv_heads * vdim)     # the gate's first column of the product
 
     def tensor_specs(self):
         H, G, D, Dv, h = self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.hidden_size
         specs = {"q": TensorSpec((H * D, h), "fan_in"), "k": TensorSpec((G * D, h), "fan_in"), "v": TensorSpec((G * Dv, h), "fan_in"),
                  "o": TensorSpec((h, H * Dv), "fan_in")}
+        if self.keys_as_values:
+            del specs["v"]
         if self.gate:
             specs["g"] = TensorSpec((H * Dv, h), "fan_in")
         if self.qk_norm == "head":
@@ -178,10 +190,8 @@ class GatedAttention(Mixer):
     def bind(self, tensors, rt):
         from .rope import rotary_frequencies
         self.rt = rt
-        parts = [tensors[n] for n in ("q", "k", "v") + (("g",) if self.gate else ())]
-        if len({p.dtype for p in parts}) > 1:
-            parts = [p.float() for p in parts]
-        self.w_in = rt.place(torch.cat(parts, 0))
+        w, _ = _padded_rows([tensors[n] for n in self.in_names + (("g",) if self.gate else ())], 1)
+        self.w_in = rt.place(w)
         self.w_o = rt.place(tensors["o"])
         small = lambda n: tensors[n].float().to(rt.device).contiguous()        # read as float32 by the kernel
         weighted = self.qk_norm and self.qk_norm != "unit"
@@ -209,11 +219,12 @@ class GatedAttention(Mixer):
             dist = tensors["rel"].float()[idx].t().to(rt.device).contiguous()         # [H, far + 1]: a head's biases side by side
         from ..kernels import ops
         self.mods = None
-        if self.softcap > 0 or self.sink or dist is not None:
+        slope = torch.tensor(self.slopes, dtype=torch.float32, device=rt.device) if self.slopes is not None else None
+        if self.softcap > 0 or self.sink or dist is not None or slope is not None:
             term = None
             if self.sink:
                 term = small("sink") if self.sink is True else torch.zeros(self.num_heads, dtype=torch.float32, device=rt.device)
-            self.mods = ops.ScoreMods(self.softcap, term, dist)
+            self.mods = ops.ScoreMods(self.softcap, term, dist, slope)
 
     def cache_need(self):
         return self.need
@@ -228,8 +239,8 @@ class GatedAttention(Mixer):
         T = ctx.num_tokens
         proj = self.rt.linear(x, self.w_in, self.b_in)
         q = self.rt.empty(T, H, DP)
-        ops.qk_norm_rope(proj, ctx.positions, ctx.slots[cache.group], self.freq, q, cache.k, cache.v, num_heads=H,
-                         num_kv_heads=G, dim=D, vdim=Dv, rot=self.rot_dims, page_size=cache.page_size, eps=self.eps,
+        ops.qk_norm_rope(proj, ctx.positions, ctx.slots[cache.group], self.freq, q, cache.k, None if self.keys_as_values else cache.v,
+                         num_heads=H, num_kv_heads=G, dim=D, vdim=Dv, rot=self.rot_dims, page_size=cache.page_size, eps=self.eps,
                          q_weight=self.q_norm, k_weight=self.k_norm, temp=self.temp, write_cache=cache.writes,
                          head_norm=self.qk_norm in ("head", "unit"), v_freq=self.v_freq, interleaved=self.rot_pairing == "interleaved", pos_temp=self.q_temp)
         heads = self.rt.empty(T, H, DP)
@@ -242,7 +253,7 @@ class GatedAttention(Mixer):
         if self.gate or DP != Dv:
             gated = self.rt.empty(T, H * Dv)
             if self.gate:
-                ops.sigmoid_gate(heads, proj[:, (H + G) * D + G * Dv:], gated, H, Dv)
+                ops.sigmoid_gate(heads, proj[:, self.gate_at:], gated, H, Dv)
             else:
                 gated.view(T, H, Dv).copy_(heads[:, :, :Dv])
         else:

@@ -64,12 +64,14 @@ def build_part(category: str, spec: PartSpec):
 class KVNeed:
     """Pages of keys and values: all positions (``window`` and ``chunk`` None), the last ``window``, or the
     positions of the newest token's own block of ``chunk`` positions (blocks counted from position 0); with a window or
-    a block, the first ``keep`` positions of the sequence are kept besides."""
+    a block, the first ``keep`` positions of the sequence are kept besides.  ``shared``: the keys serve as values too, so a
+    position is stored once (``LayerCache.k`` and ``.v`` are the same tensor)."""
     num_kv_heads: int
     head_dim: int
     window: int | None = None
     chunk: int | None = None
     keep: int = 0
+    shared: bool = False
 
     def mask(self) -> int:
         """The kernels' one integer for this need: 0 all keys, w > 0 a sliding window, -c a block of c positions."""

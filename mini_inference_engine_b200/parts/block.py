@@ -5,7 +5,7 @@ is fused into the *next* norm, so a block takes the pending ``delta`` and return
 add+norm, after the last layer into the final norm)."""
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 
 from ..weights.loader import TensorSpec
 from ..kernels import ops
@@ -95,6 +95,84 @@ class Branches:
         self.deltas, self.inner_weights, self.coef = tuple(deltas), tuple(inner_weights), coef
         self.coefs = tuple(coefs) if coefs is not None else None      # a coefficient per output instead of one for the sum
         self.scaled = scaled            # (h [T, W], w float32 [T]): one more output, w[t] * h[t] (norms that add by ``add_to``)
+
+
+@dataclass
+class NormedDelta:
+    """What a block leaves for the next reader of the stream when the sublayer's output is normed before it is added: the output ``y``
+    (a tensor or ``Branches``; None: nothing), the ``norm`` that belongs to it, and what else is to be added before the reader:
+    ``extra`` (float32, of the stream's shape) and ``shift`` (float32 [width])."""
+    y: object = None
+    norm: object = None
+    extra: object = None
+    shift: object = None
+
+
+class SandwichResidual(Block):
+    """Norms before and after each sublayer: x <- x + mixer_out_norm(mixer(mixer_norm(x))), then the same with the feed-forward, which
+    may be absent.  A constant on the branches is the out-norms' ``gain``.  The out-norm, the sum and the next norm are one kernel, so a
+    block takes and returns a ``NormedDelta``."""
+    roles = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "mixer_out_norm": "norm", "feed_forward_norm": "norm",
+             "feed_forward_out_norm": "norm"}
+    optional_roles = ("feed_forward", "feed_forward_norm", "feed_forward_out_norm")
+
+    def __init__(self, **parts):
+        super().__init__(**parts)
+        if len({r in parts for r in self.optional_roles}) != 1:
+            raise ValueError("a feed-forward comes with both of its norms, and they with it")
+
+    def forward(self, delta, res, ctx, cache):
+        pending = NormedDelta(self.mixer.forward(self.mixer_norm(delta, res), ctx, cache), self.mixer_out_norm)
+        if getattr(self, "feed_forward", None) is None:
+            return pending
+        return NormedDelta(self.feed_forward.forward(self.feed_forward_norm(pending, res), ctx), self.feed_forward_out_norm)
+
+
+register_part("block", "sandwich_residual", SandwichResidual)
+
+
+class StreamShift(Part):
+    """A vector added to the stream, and the embedding's output e with it where ``with_embedding`` says so (the embedding keeps it,
+    ``ctx.extras["embedding_output"]``): x <- x + e + b with b = row ``index`` of 'step' [rows, width].  Models that run a stretch of
+    layers several times put one in front of every pass, all sharing the tensor.  Nothing is computed here: both ride on
+    what is pending into the next norm's kernel."""
+
+    def __init__(self, hidden_size: int, rows: int, index: int, with_embedding: bool):
+        if not 0 <= index < rows:
+            raise ValueError(f"shift {index} of {rows}")
+        self.hidden_size, self.rows, self.index, self.with_embedding = hidden_size, rows, index, bool(with_embedding)
+
+    def tensor_specs(self):
+        return {"step": TensorSpec((self.rows, self.hidden_size), "normal:0:0.1")}
+
+    def bind(self, tensors, rt):
+        self.rt = rt
+        self.shift = tensors["step"][self.index].float().to(rt.device).contiguous()
+
+    def pending(self, delta, ctx):
+        extra = None
+        if self.with_embedding:
+            extra = ctx.extras.get("embedding_output")
+            if extra is None:
+                raise ValueError("adding the embedding's output needs an embedding that keeps it (keep_output)")
+        d = delta if delta is not None else NormedDelta()
+        if not isinstance(d, NormedDelta) or d.shift is not None:
+            raise ValueError("a shift of the stream rides on a NormedDelta, one at a time")
+        return replace(d, extra=extra, shift=self.shift)
+
+
+register_part("connection", "stream_shift", StreamShift)
+
+
+class StreamShiftStep(Block):
+    """Not a layer but a step between layers: its one part adds to what is pending (``StreamShift``)."""
+    roles = {"shift": "connection"}
+
+    def forward(self, delta, res, ctx, cache):
+        return self.shift.pending(delta, ctx)
+
+
+register_part("block", "stream_shift_step", StreamShiftStep)
 
 
 class StreamMix(Part):

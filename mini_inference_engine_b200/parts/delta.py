@@ -67,7 +67,10 @@ class ChannelDelta(Mixer):
         up[H * D:, ra:ra + rg] = g2
         self.w_up = rt.place(up)
         self.w_o = rt.place(tensors["o"])
-        small = lambda t: t.float().to(rt.device).contiguous()               # read as float32 by the kernels
+        self.bind_small(tensors)
+
+    def bind_small(self, tensors):
+        small = lambda t: t.float().to(self.rt.device).contiguous()          # read as float32 by the kernels
         self.conv = small(torch.cat([tensors["q.conv"].float(), tensors["k.conv"].float(), tensors["v.conv"].float()], 0))
         self.a_log, self.dt_bias, self.norm = small(tensors["A_log"]), small(tensors["dt_bias"]), small(tensors["norm"])
 
@@ -98,3 +101,52 @@ class ChannelDelta(Mixer):
 
 
 register_part("mixer", "channel_delta", ChannelDelta)
+
+
+class HeadDelta(ChannelDelta):
+    """The gated delta rule with ONE decay per head, g = exp(-exp(A_log_h) softplus(W_a h + dt_bias)_h), and an output gate silu(W_g h) laid
+    out heads x vdim; everything else as ``ChannelDelta``.  q|k|v|g of the input are one product; a|b, which decide decays and
+    step sizes, a second one that leaves float32."""
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, taps: int, eps: float, unit_eps: float = 1e-6):
+        super().__init__(hidden_size, num_heads, num_kv_heads, dim, vdim, taps, eps, unit_eps=unit_eps)
+
+    def tensor_specs(self):
+        H, Dv, h = self.num_heads, self.vdim, self.hidden_size
+        specs = {n: s for n, s in super().tensor_specs().items() if n not in ("a1", "a2", "g1", "g2")}
+        specs.update({"a": TensorSpec((H, h), "fan_in"), "dt_bias": TensorSpec((H,), "uniform:-4:1"), "g": TensorSpec((H * Dv, h), "fan_in")})
+        return specs
+
+    def bind(self, tensors, rt):
+        self.rt = rt
+        w, _ = _padded_rows([tensors[n] for n in ("q", "k", "v", "g")])
+        self.w_in = rt.place(w)
+        w, _ = _padded_rows([tensors["a"], tensors["b"]])
+        self.w_gates = rt.place(w)
+        self.w_o = rt.place(tensors["o"])
+        self.bind_small(tensors)
+
+    def kernel_sources(self):
+        return {"delta_rule"} | self.rt.product_sources(self.w_in, self.w_gates, self.w_o)
+
+    def forward(self, x, ctx, cache):
+        H, G, D, Dv, T = self.num_heads, self.num_kv_heads, self.dim, self.vdim, ctx.num_tokens
+        state, conv_state = cache.parts[0].state, cache.parts[1].state
+        proj = self.rt.linear(x, self.w_in)
+        gates = self.rt.linear(x, self.w_gates, None, out_dtype=torch.float32)               # [a: H | b: H]
+        f32 = lambda n: self.rt.empty(T, n, dtype=torch.float32)
+        qn, kn, vn, beta, decay, kq = f32(G * D), f32(G * D), f32(H * Dv), f32(H), f32(H), f32(G)
+        ops.delta_prepare(proj, gates, self.conv, conv_state, ctx.token_row, ctx.row_q_start, ctx.state_slots, self.a_log, self.dt_bias,
+                          qn, kn, vn, beta, decay, kq, num_heads=H, num_kv_heads=G, dim=D, vdim=Dv, unit_eps=self.unit_eps, per_head=True)
+        if self.taps > 1:
+            ops.conv_state_update(proj, ctx.row_q_start, ctx.row_q_len, ctx.state_slots, conv_state)
+        o = f32(H * Dv)
+        ops.delta_scan(qn, kn, vn, beta, decay, kq, ctx.row_q_start, ctx.row_q_len, ctx.state_slots, state, o, num_heads=H,
+                       num_kv_heads=G, dim=D, vdim=Dv)
+        gated = self.rt.empty(T, H * Dv)
+        at = 2 * G * D + H * Dv
+        ops.head_norm_gate(o, proj[:, at:at + H * Dv], self.norm, gated, H, Dv, self.eps, silu=True)
+        return self.rt.linear(gated, self.w_o, None, out_dtype=torch.float32)
+
+
+register_part("mixer", "head_delta", HeadDelta)

@@ -85,6 +85,51 @@ class LayerNorm(Part):
 register_part("norm", "layernorm", LayerNorm)
 
 
+class ZeroCenteredRMSNorm(Part):
+    """RMS norm whose weight is stored around zero: x / sqrt(mean(x^2) + eps) * (1 + w) * ``gain``.  It serves both ends of a
+    sublayer: called like the other norms (``norm(delta, res, rows)``) it norms the stream for a reader, after adding what is pending --
+    a ``NormedDelta``: the output of the sublayer before, normed by a norm of this kind (whose ``gain`` is the constant on the
+    branch), and what comes between two layers; sum, both norms and the stream's update are one kernel.  The gain of a norm in
+    front of the output head is a factor on the logits."""
+
+    def __init__(self, size: int, eps: float, gain: float = 1.0):
+        self.size, self.eps, self.gain = size, eps, float(gain)
+
+    def tensor_specs(self):
+        return {"weight": TensorSpec((self.size,), "normal:0:0.1")}
+
+    def bind(self, tensors, rt):
+        self.rt = rt
+        self.weight = ((1.0 + tensors["weight"].double()) * self.gain).float().to(rt.device).contiguous()      # the factor itself, float32
+
+    def kernel_sources(self):
+        return {"sandwich_norm"}
+
+    def __call__(self, delta, res, rows=None):
+        n_out = rows.numel() if rows is not None else res.shape[0]
+        out = self.rt.empty(n_out, self.size)
+        return apply_pending(delta, res, self.eps, weight=self.weight, out=out, rows=rows)
+
+
+def apply_pending(delta, res, eps: float, **reader):
+    """Adds a ``NormedDelta`` (or nothing) to the stream, in one kernel with the norm of ``reader`` (``ops.sandwich_norm``'s weight, out
+    and rows) where one is given."""
+    from .block import NormedDelta
+    if delta is None:
+        return ops.sandwich_norm(res, eps, **reader)
+    if not isinstance(delta, NormedDelta):
+        raise ValueError("this norm takes the output of the sublayer before together with the norm that belongs to it (NormedDelta)")
+    norm = delta.norm
+    if norm is not None and norm.eps != eps:
+        raise ValueError(f"the norms on both sides of the stream share an eps; got {norm.eps} and {eps}")
+    deltas, coefs = addends_of(delta.y)
+    return ops.sandwich_norm(res, eps, deltas=deltas, coefs=coefs, delta_weight=norm.weight if norm is not None else None, extra=delta.extra,
+                             shift=delta.shift, **reader)
+
+
+register_part("norm", "zero_centered_rmsnorm", ZeroCenteredRMSNorm)
+
+
 class GroupRMSNorm(Part):
     """RMS norm with statistics per group: a row is cut into ``groups`` equal consecutive parts, each divided by
     sqrt(mean(part^2) + eps), and the whole multiplied by the weight.  It norms the stream itself (post-norm
