@@ -490,12 +490,29 @@ def radenex_configs(size: dict, vocab=32000, positions=4096):
     return radenex, design_configs(size, vocab, positions)[1]
 
 
+def karopel_configs(size: dict, vocab=32000, positions=4096):
+    """A Karopel configuration of the given layer sizes -- keys-as-values attention with a window of 1,024 beside a gated delta rule,
+    windowed attention that keeps the first 64 tokens, and the first kind again, as a stretch that runs twice: six layer runs with
+    Llama's silu-gated feed-forward -- and the Llama configuration with the same width, heads and number of layers."""
+    from mini_inference_engine_b200.config import load_config
+    w, ff, H, G = size["width"], size["ff"], size["heads"], size["kv_heads"]
+    mlp = dict(kind="dense", ff=ff)
+    par = dict(type="parallel", mlp=mlp, mixer=dict(left_scale=1.0, right_scale=1.0,
+               left=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024)),
+               right=dict(heads=H, kv_heads=H // 2, dim=128, vdim=128, conv=4)))
+    win = dict(type="attention", mlp=mlp, mixer=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024, keep_first=64),
+                                                     rot=dict(base=5e5, dims=128, scaling=dict(factor=8.0, low=1.0, high=4.0, original=positions))))
+    karopel = load_config(dict(architecture="Karopel", vocab=vocab, width=w, norm=dict(eps=1e-5), residual_mult=0.5, logit_scale=0.25,
+                               loop=dict(start=0, stop=3, times=2), layers=[par, win, par]))
+    return karopel, design_configs(size, vocab, positions)[1]
+
+
 KERNEL_FACES = ("embedding", "add_rmsnorm", "stream_norm", "rope_cache_write", "qk_norm_rope", "paged_attention", "prefill_attention",
                 "prefill_attention_tc", "decode_attention", "retention_scan", "head_rms_gate", "causal_conv", "recurrence_gates",
                 "recurrence_scan", "swiglu", "glu_clamped", "sigmoid_gate", "hyper_norm", "latent_norm_rope", "latent_assemble",
                 "diff_combine", "delta_prepare", "conv_state_update", "delta_scan", "head_norm_gate", "moe_route", "moe_router", "moe_dense_act", "moe_pairs", "moe_sort", "moe_gather", "moe_act_rows", "moe_combine", "grouped_linear",
                 "pair_embedding", "normed_add", "xielu", "gelu_gate_rows", "moe_glu", "add_layernorm", "stream_join", "tanh_cap",
-                "decay_scan", "gate_scan", "group_norm_gate", "turn_heads", "relu2")
+                "decay_scan", "gate_scan", "group_norm_gate", "turn_heads", "relu2", "sandwich_norm")
 
 
 class KernelTimes:
@@ -551,7 +568,7 @@ def run_design(args, steps, warmup):
     from mini_inference_engine_b200.weights import write_model_folder
     pk = peaks()
     configs_for = {"getizen": design_configs, "kebudra": kebudra_configs, "serotar": serotar_configs, "luluzen": luluzen_configs,
-                   "radenex": radenex_configs}[args.design]
+                   "radenex": radenex_configs, "karopel": karopel_configs}[args.design]
     out = {"metric": "design_comparison", "design": args.design.capitalize(), "beside": "Llama", "dtype": "bf16", "data": "synthetic (random weights, seed 0)",
            "peaks": pk, "sizes": {}}
     batches = [int(b) for b in args.points.split(",") if b] or [8]
@@ -617,7 +634,7 @@ def main():
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the configuration has (named in config)")
     ap.add_argument("--preset", default="tinyllama-1.1b")
     ap.add_argument("--points", default="1,64", help="further decode batch sizes, comma separated ('' for none)")
-    ap.add_argument("--design", default=None, choices=["getizen", "kebudra", "serotar", "luluzen", "radenex"],
+    ap.add_argument("--design", default=None, choices=["getizen", "kebudra", "serotar", "luluzen", "radenex", "karopel"],
                     help="instead of the default workload: prefill and decode throughput of this design beside Llama at equal "
                          "layer sizes (--sizes), random weights; decode batches from --points")
     ap.add_argument("--sizes", default="w2048,w4096", help="with --design: layer sizes to measure, of " + ", ".join(DESIGN_SIZES))
