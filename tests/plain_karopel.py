@@ -22,12 +22,23 @@ The design in this file's notation (t: token index = position, x_t: residual str
                      g = exp(-exp(A_log) softplus(Wa h + dt_bias)) per head; o / rms(o) * w * silu(Wg h); Wo
   feed-forward       Wd (silu(Wgate h) * (Wup h))
   head               logits = W_head n(x; w_final) * logit_scale
+
+``rnd`` (default: nothing) is applied where an implementation in 16 bits rounds -- operands and results of matrix products, heads before
+and after attention -- so that a run with it shows how much rounding alone moves each row of logits.
 """
 from __future__ import annotations
 
 import math
 
 import torch
+
+
+def exact(z: torch.Tensor) -> torch.Tensor:
+    return z
+
+
+def to_bf16(z: torch.Tensor) -> torch.Tensor:
+    return z.to(torch.bfloat16).to(z.dtype)
 
 
 def over_rms(v: torch.Tensor, eps: float) -> torch.Tensor:
@@ -113,23 +124,23 @@ def softmax_heads(q, k, v, scale: float, seen, sink=None, slope=None) -> torch.T
     return out
 
 
-def attention(h, W, p, m, eps):
+def attention(h, W, p, m, eps, rnd=exact):
     T, H, G, D, Dv = h.shape[0], int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
     pos = torch.arange(T)
-    q = over_rms((h @ W[p + "q"].T).reshape(T, H, D), eps) * W[p + "q.norm"]
-    k = over_rms((h @ W[p + "k"].T).reshape(T, G, D), eps) * W[p + "k.norm"]
-    v = (h @ W[p + "v"].T).reshape(T, G, Dv)
+    q = over_rms(rnd(h @ W[p + "q"].T).reshape(T, H, D), eps) * W[p + "q.norm"]
+    k = over_rms(rnd(h @ W[p + "k"].T).reshape(T, G, D), eps) * W[p + "k.norm"]
+    v = rnd(h @ W[p + "v"].T).reshape(T, G, Dv)
     f = speeds(m["rot"])
-    o = softmax_heads(turn_neighbours(q, pos, f), turn_neighbours(k, pos, f), v, float(m["scale"]), visible(T, m.get("mask")), sink=W[p + "sink"])
-    return o.reshape(T, H * Dv) @ W[p + "o"].T
+    o = softmax_heads(rnd(turn_neighbours(q, pos, f)), rnd(turn_neighbours(k, pos, f)), v, float(m["scale"]), visible(T, m.get("mask")), sink=W[p + "sink"])
+    return rnd(o.reshape(T, H * Dv)) @ W[p + "o"].T
 
 
-def keys_as_values(h, W, p, m, eps):
+def keys_as_values(h, W, p, m, eps, rnd=exact):
     T, H, G, D = h.shape[0], int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
-    q = (h @ W[p + "q"].T).reshape(T, H, D)
-    k = (h @ W[p + "k"].T).reshape(T, G, D)
+    q = rnd(h @ W[p + "q"].T).reshape(T, H, D)
+    k = rnd(h @ W[p + "k"].T).reshape(T, G, D)
     o = softmax_heads(q, k, k, float(m["scale"]), visible(T, m.get("mask")), slope=slopes(H))
-    return o.reshape(T, H * D) @ W[p + "o"].T
+    return rnd(o.reshape(T, H * D)) @ W[p + "o"].T
 
 
 # --------------------------------------------------------------------------- gated delta rule
@@ -154,28 +165,28 @@ def delta_steps(q, k, v, beta, g):
     return torch.stack(out)
 
 
-def gated_delta(h, W, p, m, eps):
+def gated_delta(h, W, p, m, eps, rnd=exact):
     T, H, G, D, Dv = h.shape[0], int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
-    q, k, v = (short_convolution(h @ W[p + n].T, W[p + n + ".conv"]) for n in "qkv")
+    q, k, v = (short_convolution(rnd(h @ W[p + n].T), W[p + n + ".conv"]) for n in "qkv")
     unit = lambda z: z / torch.sqrt((z * z).sum(-1, keepdim=True) + 1e-6)
     q, k = unit(q.reshape(T, G, D)) * D ** -0.5, unit(k.reshape(T, G, D))
     q, k = (z.repeat_interleave(H // G, 1) for z in (q, k))
     beta = torch.sigmoid(h @ W[p + "b"].T)
     g = torch.exp(-torch.exp(W[p + "A_log"]) * softplus(h @ W[p + "a"].T + W[p + "dt_bias"]))
     o = over_rms(delta_steps(q, k, v.reshape(T, H, Dv), beta, g), eps) * W[p + "norm"]
-    return (o.reshape(T, H * Dv) * silu(h @ W[p + "g"].T)) @ W[p + "o"].T
+    return rnd(o.reshape(T, H * Dv) * silu(rnd(h @ W[p + "g"].T))) @ W[p + "o"].T
 
 
-def parallel(h, W, p, m, eps):
-    return (float(m["left_scale"]) * keys_as_values(h, W, p + "left.", m["left"], eps)
-            + float(m["right_scale"]) * gated_delta(h, W, p + "right.", m["right"], eps))
+def parallel(h, W, p, m, eps, rnd=exact):
+    return (float(m["left_scale"]) * keys_as_values(h, W, p + "left.", m["left"], eps, rnd)
+            + float(m["right_scale"]) * gated_delta(h, W, p + "right.", m["right"], eps, rnd))
 
 
 MIXERS = {"attention": attention, "parallel": parallel}
 
 
-def feed_forward(h, W, p):
-    return (silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
+def feed_forward(h, W, p, rnd=exact):
+    return rnd(silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
 
 
 # --------------------------------------------------------------------------- the model
@@ -198,23 +209,23 @@ def before_pass(x, e, W, t: int):
     return x + W["loop.step"][t]
 
 
-def layer(x, W, p, spec, eps, m):
-    y = MIXERS[spec["type"]](norm_about_one(x, W[p + "norm1"], eps), W, p + "mix.", spec["mixer"], eps)
+def layer(x, W, p, spec, eps, m, rnd=exact):
+    y = MIXERS[spec["type"]](rnd(norm_about_one(x, W[p + "norm1"], eps)), W, p + "mix.", spec["mixer"], eps, rnd)
     x = x + m * norm_about_one(y, W[p + "norm1b"], eps)
     if spec.get("mlp") is not None:
-        y = feed_forward(norm_about_one(x, W[p + "norm2"], eps), W, p + "mlp.")
+        y = feed_forward(rnd(norm_about_one(x, W[p + "norm2"], eps)), W, p + "mlp.", rnd)
         x = x + m * norm_about_one(y, W[p + "norm2b"], eps)
     return x
 
 
-def forward(cfg: dict, W: dict, tokens, trace: list | None = None) -> torch.Tensor:
+def forward(cfg: dict, W: dict, tokens, trace: list | None = None, rnd=exact) -> torch.Tensor:
     """Logits [T, vocab]; ``trace`` collects the stream after every layer run."""
     eps, m = float(cfg["norm"]["eps"]), float(cfg.get("residual_mult", 1.0))
     x = e = W["embed"][torch.as_tensor(list(tokens))]
     for i, t in run_order(cfg):
         if t is not None:
             x = before_pass(x, e, W, t)
-        x = layer(x, W, f"l{i}.", cfg["layers"][i], eps, m)
+        x = layer(x, W, f"l{i}.", cfg["layers"][i], eps, m, rnd)
         if trace is not None:
             trace.append(x)
-    return (norm_about_one(x, W["final.norm"], eps) @ W["head"].T) * float(cfg.get("logit_scale", 1.0))
+    return (rnd(norm_about_one(x, W["final.norm"], eps)) @ W["head"].T) * float(cfg.get("logit_scale", 1.0))
