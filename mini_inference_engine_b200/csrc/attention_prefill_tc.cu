@@ -104,7 +104,8 @@ __device__ __forceinline__ float ex2_approx(float x) {
 }
 
 // MODS: what scores pass between the product and the softmax (ScoreMods): bit 0 a cap, bit 1 a bias by distance, bit 2
-// a slope by distance (alone); an instance for each combination, so that the plain softmax keeps its instruction count and the others test nothing per element.  A sink
+// a slope by distance (alone; key tiles then go from the query backwards, so that the largest scores come first and the running
+// maximum settles); an instance for each combination, so that the plain softmax keeps its instruction count and the others test nothing per element.  A sink
 // joins the sum in every instance (it costs a term at a row's start).  KEEP: the instance for a window or block that keeps the
 // first keys in sight (p.keep).
 template <int D, int MODS, bool KEEP>
@@ -227,6 +228,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
             }
             auto key0_of = [&](int g) {
                 const int t = g < nA ? g : g - nA, kept = g < nA ? sb[0].kept : sb[1].kept;
+                if (MODS & 4) return (g < nA ? sb[0].kbeg + (nA - 1) * FA_BN : sb[1].kbeg + (G - nA - 1) * FA_BN) - t * FA_BN;
                 return t < kept ? t * FA_BN : (g < nA ? sb[0].kbeg : sb[1].kbeg) + (t - kept) * FA_BN;
             };
             auto copies_of = [&](int g) {
@@ -374,7 +376,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,   // qkv 
                     ok = __all_sync(0xffffffffu, mbar_wait(&s_full, g & 1, abort_p));     // the warp goes on or gives up as one
                     if (!ok) break;
                     tc_fence_after();
-                    const int key0 = t < kept ? t * FA_BN : kbeg + (t - kept) * FA_BN;
+                    const int key0 = (MODS & 4) ? kbeg + (ntiles - 1 - t) * FA_BN : t < kept ? t * FA_BN : kbeg + (t - kept) * FA_BN;
                     // masks are needed only where the tile touches the diagonal, the window's edge or the range's start
                     bool need_mask = key0 + FA_BN - 1 > pos0 || key0 < k_lo || (p.window != 0 && key0 < mask_first_key(pos0 + FA_BM - 1, p.window));
                     // A key is read if lo <= key <= hi or, with kept keys, if it is below `also`: a tile in front of the window's holds kept

@@ -47,7 +47,8 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int64_t stride,
                                      const int* __restrict__ state_slots, const float* __restrict__ a_log,
                                      const float* __restrict__ dt_bias, float* __restrict__ qn, float* __restrict__ kn,
                                      float* __restrict__ vn, float* __restrict__ beta, float* __restrict__ decay,
-                                     float* __restrict__ kq, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps, int per_head) {
+                                     float* __restrict__ kq, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps, int per_head,
+                                     float* __restrict__ log_decay) {
     pdl_enter();
     const int t = blockIdx.x, A = per_head ? 1 : D;
     const int row = token_row[t];
@@ -96,8 +97,10 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int64_t stride,
         beta[(int64_t)t * H + h] = 1.0f / (1.0f + expf(-z));
     }
     for (int i = threadIdx.x; i < H * A; i += blockDim.x) {
-        const float rate = expf(a_log[i / A]);
-        decay[(int64_t)t * H * A + i] = expf(-rate * softplus_f(lo[i] + dt_bias[i]));
+        const float rate = expf(a_log[i / A]), ld = -rate * softplus_f(lo[i] + dt_bias[i]);
+        decay[(int64_t)t * H * A + i] = expf(ld);
+        // (e^-100 is nothing in 32 bits; the bound keeps sums of log decays, and their differences, exact to a few parts in a million)
+        if (log_decay) log_decay[(int64_t)t * H * A + i] = fmaxf(ld, -100.f);
     }
     __syncthreads();                                   // q and k of this token, written above by other warps of the block
     for (int g = warp; g < G; g += nw) {               // k . q per key head: the same for every value column of the recurrence
@@ -153,7 +156,7 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
                                   const float* __restrict__ beta, const float* __restrict__ decay, const float* __restrict__ kq,
                                   const int* __restrict__ row_q_start, const int* __restrict__ row_q_len,
                                   const int* __restrict__ state_slots, float* __restrict__ state, float* __restrict__ out, int H,
-                                  int G, int D, int Dv, int L_rt, int cols, int tb, int slot_floats) {
+                                  int G, int D, int Dv, int L_rt, int cols, int tb, int slot_floats, int below) {
     extern __shared__ __align__(16) float ring[];
     pdl_enter();
     const int L = LT > 0 ? LT : L_rt;                         // lanes a column: a constant where the launcher knows it (shifts, unrolled sums)
@@ -161,6 +164,7 @@ __global__ void delta_scan_kernel(const float* __restrict__ qn, const float* __r
     const int l = threadIdx.x % L, cl = threadIdx.x / L, j0 = blockIdx.z * cols, j = j0 + cl;
     const bool active = cl < cols && j < Dv;                   // threads that only fill up the last warp own no column
     const int n = row_q_len[row], t0 = row_q_start[row];
+    if (n >= below) return;                                    // a row that another kernel serves (delta_chunk.cu)
     const int kh = h / (H / G);
     float* sp = state + (((int64_t)state_slots[row] * H + h) * Dv + (active ? j : 0)) * D;
     // register r of lane l holds row 4 (l + L (r / 4)) + r % 4: pieces of four consecutive rows, dealt out over the lanes,
@@ -345,7 +349,7 @@ extern "C" int mie_delta_prepare(const void* proj, int tag, long long stride, co
                                  const float* conv_state, const int* token_row, const int* row_q_start, const int* state_slots,
                                  const float* a_log, const float* dt_bias, float* qn, float* kn, float* vn, float* beta, float* decay,
                                  float* kq, int num_tokens, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps, int per_head,
-                                 cudaStream_t stream) {
+                                 float* log_decay, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || K < 1) return MIE_ERR_BAD_ARG;
     const int units = 2 * G + H;
@@ -353,11 +357,11 @@ extern "C" int mie_delta_prepare(const void* proj, int tag, long long stride, co
     if (tag == MIE_F32)
         return launch_kernel(delta_prepare_kernel<float>, dim3(num_tokens), dim3(threads), 0, stream, (const float*)proj, (int64_t)stride,
                              low, (int64_t)low_stride, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias, qn, kn, vn,
-                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps, per_head);
+                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps, per_head, log_decay);
     else if (tag == MIE_BF16)
         return launch_kernel(delta_prepare_kernel<bf16>, dim3(num_tokens), dim3(threads), 0, stream, (const bf16*)proj, (int64_t)stride,
                              low, (int64_t)low_stride, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias, qn, kn, vn,
-                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps, per_head);
+                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps, per_head, log_decay);
     return MIE_ERR_BAD_ARG;
 }
 
@@ -379,7 +383,7 @@ extern "C" int mie_conv_state_update(const void* x, int tag, long long stride, c
 template <int R, bool ONE>
 static int launch_scan(const float* qn, const float* kn, const float* vn, const float* beta, const float* decay, const float* kq,
                        const int* row_q_start, const int* row_q_len, const int* state_slots, float* state, float* out, int num_rows,
-                       int H, int G, int D, int Dv, cudaStream_t stream) {
+                       int H, int G, int D, int Dv, int below, cudaStream_t stream) {
     int L = 1;
     while (L * R < D) L <<= 1;
     if (L > 32) return MIE_ERR_TOO_LARGE;
@@ -403,17 +407,17 @@ static int launch_scan(const float* qn, const float* kn, const float* vn, const 
         if (e != cudaSuccess) return (int)e;
     }
     return launch_kernel(kernel, grid, dim3(threads), smem, stream, qn, kn, vn, beta, decay, kq, row_q_start, row_q_len,
-                         state_slots, state, out, H, G, D, Dv, L, cols, tb, slot_floats);
+                         state_slots, state, out, H, G, D, Dv, L, cols, tb, slot_floats, below);
 }
 
 extern "C" int mie_delta_scan(const float* qn, const float* kn, const float* vn, const float* beta, const float* decay, const float* kq,
                               const int* row_q_start, const int* row_q_len, const int* state_slots, float* state, float* out,
-                              int num_rows, int H, int G, int D, int Dv, int A, cudaStream_t stream) {
+                              int num_rows, int H, int G, int D, int Dv, int A, int below, cudaStream_t stream) {
     if (num_rows <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || (A != 1 && A != D)) return MIE_ERR_BAD_ARG;
     // entries of a column a lane: the fewest for which sixteen lanes hold a column (thirty-two for the longest keys)
-#define SCAN(R) (A == 1 ? launch_scan<R, true>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, stream)  \
-                        : launch_scan<R, false>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, stream))
+#define SCAN(R) (A == 1 ? launch_scan<R, true>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, below, stream)  \
+                        : launch_scan<R, false>(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, num_rows, H, G, D, Dv, below, stream))
     if (D <= 64) return SCAN(4);
     if (D <= 128) return SCAN(8);
     if (D <= DELTA_MAX_KEY) return SCAN(16);

@@ -1184,12 +1184,13 @@ def diff_combine(maps: torch.Tensor, gate, out: torch.Tensor, *, num_heads: int,
 
 def delta_prepare(proj: torch.Tensor, low: torch.Tensor, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias,
                   qn, kn, vn, beta, decay, kq, *, num_heads: int, num_kv_heads: int, dim: int, vdim: int, unit_eps: float,
-                  per_head: bool = False) -> None:
+                  per_head: bool = False, log_decay=None) -> None:
     """From rows [q: G x dim | k: G x dim | v: H x vdim | beta logits: H | ...] of the input projection and float32 rows
     [a: H x dim | ...] of the low-rank one: convolution over time + silu of q, k, v (float32 taps [channels, K], older inputs
     from ``conv_state`` [slots, K - 1, channels]), q and k unit vectors per head (q times dim^-1/2), beta = sigmoid,
     decay = exp(-exp(a_log[h]) softplus(a + dt_bias)), kq = k . q per key head.  All outputs float32.  ``per_head``: one decay per head (``decay`` [T, H]);
-    the float32 rows are [a: H | beta logits: H | ...] and the projection's hold q, k and v only."""
+    the float32 rows are [a: H | beta logits: H | ...] and the projection's hold q, k and v only.  ``log_decay``: the decays'
+    logarithms too, none below -100 (float32, of ``decay``'s shape)."""
     T = proj.shape[0]
     H, G, D, Dv = num_heads, num_kv_heads, dim, vdim
     C = 2 * G * D + H * Dv
@@ -1211,7 +1212,7 @@ def delta_prepare(proj: torch.Tensor, low: torch.Tensor, taps, conv_state, token
     _check(lib.mie_delta_prepare(_ptr(proj), tag(proj), ctypes.c_longlong(proj.stride(0)), _ptr(low), ctypes.c_longlong(low.stride(0)),
                                  _ptr(taps), _ptr(conv_state), _ptr(token_row), _ptr(row_q_start), _ptr(state_slots), _ptr(a_log),
                                  _ptr(dt_bias), _ptr(qn), _ptr(kn), _ptr(vn), _ptr(beta), _ptr(decay), _ptr(kq), T, H, G, D, Dv, K,
-                                 ctypes.c_float(D ** -0.5), ctypes.c_float(unit_eps), int(per_head), _stream()), "delta_prepare")
+                                 ctypes.c_float(D ** -0.5), ctypes.c_float(unit_eps), int(per_head), _ptr(log_decay), _stream()), "delta_prepare")
 
 
 def conv_state_update(x: torch.Tensor, row_q_start, row_q_len, state_slots, conv_state) -> None:
@@ -1228,9 +1229,10 @@ def conv_state_update(x: torch.Tensor, row_q_start, row_q_len, state_slots, conv
 
 
 def delta_scan(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots, state, out, *, num_heads: int, num_kv_heads: int,
-               dim: int, vdim: int) -> torch.Tensor:
+               dim: int, vdim: int, below: int = 1 << 30) -> torch.Tensor:
     """S <- decay S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q for every new token of every row, from and to
-    ``state`` [slots, H, vdim, dim] float32.  ``decay`` [T, H * dim], or [T, H]: one per head.  ``out`` [T, H * vdim] float32."""
+    ``state`` [slots, H, vdim, dim] float32.  ``decay`` [T, H * dim], or [T, H]: one per head.  ``out`` [T, H * vdim] float32.  Rows with
+    ``below`` new tokens or more are left alone (``delta_chunks``)."""
     T = qn.shape[0]
     H, G, D, Dv = num_heads, num_kv_heads, dim, vdim
     A = decay.shape[1] // H
@@ -1242,7 +1244,34 @@ def delta_scan(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots,
         _i32(t, n)
     lib = load("delta_rule")
     _check(lib.mie_delta_scan(_ptr(qn), _ptr(kn), _ptr(vn), _ptr(beta), _ptr(decay), _ptr(kq), _ptr(row_q_start), _ptr(row_q_len),
-                              _ptr(state_slots), _ptr(state), _ptr(out), row_q_len.numel(), H, G, D, Dv, A, _stream()), "delta_scan")
+                              _ptr(state_slots), _ptr(state), _ptr(out), row_q_len.numel(), H, G, D, Dv, A, int(below), _stream()), "delta_scan")
+    return out
+
+
+def delta_chunks_take(dim: int) -> bool:
+    """Whether ``delta_chunks`` serves keys of this size."""
+    return dim % 4 == 0 and dim <= 128
+
+
+def delta_chunks(qn, kn, vn, beta, log_decay, row_q_start, row_q_len, state_slots, state, out, *, num_heads: int, num_kv_heads: int, dim: int,
+                 vdim: int, min_len: int, work=None) -> torch.Tensor:
+    """``delta_scan`` with one decay per head, in chunks of 64 tokens, for the rows with ``min_len`` new tokens or more (the others are left
+    alone).  ``log_decay`` [T, H] float32, not positive.  ``work`` = (rows, tokens) of those rows where the caller knows."""
+    T = qn.shape[0]
+    H, G, D, Dv = num_heads, num_kv_heads, dim, vdim
+    _need(delta_chunks_take(D), f"keys of {D}: the chunked kernel takes multiples of 4 up to 128")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, Dv, D), "state must be float32 [slots, H, vdim, dim]")
+    for t, n in ((qn, G * D), (kn, G * D), (vn, H * Dv), (beta, H), (log_decay, H), (out, H * Dv)):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n), "operands must be float32 [T, n]")
+    for t, n in ((row_q_start, "row_q_start"), (row_q_len, "row_q_len"), (state_slots, "state_slots")):
+        _i32(t, n)
+    lib = load("delta_chunk")
+    rows, tokens = work if work is not None else (row_q_len.numel(), T)
+    size = lib.mie_delta_chunk_tokens()
+    chunks = tokens // size + min(rows, tokens // max(1, min_len))
+    scratch = _workspace(qn.device, "delta_chunks", chunks * H * lib.mie_delta_chunk_floats(), torch.float32)
+    _check(lib.mie_delta_chunks(_ptr(qn), _ptr(kn), _ptr(vn), _ptr(beta), _ptr(log_decay), _ptr(row_q_start), _ptr(row_q_len), _ptr(state_slots),
+                                _ptr(state), _ptr(out), _ptr(scratch), chunks, row_q_len.numel(), int(min_len), H, G, D, Dv, _stream()), "delta_chunks")
     return out
 
 

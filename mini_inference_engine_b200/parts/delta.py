@@ -103,6 +103,9 @@ class ChannelDelta(Mixer):
 register_part("mixer", "channel_delta", ChannelDelta)
 
 
+CHUNKED_FROM = 40        # new tokens from which a row's recurrence goes in chunks
+
+
 class HeadDelta(ChannelDelta):
     """The gated delta rule with ONE decay per head, g = exp(-exp(A_log_h) softplus(W_a h + dt_bias)_h), and an output gate silu(W_g h) laid
     out heads x vdim; everything else as ``ChannelDelta``.  q|k|v|g of the input are one product; a|b, which decide decays and
@@ -127,7 +130,7 @@ class HeadDelta(ChannelDelta):
         self.bind_small(tensors)
 
     def kernel_sources(self):
-        return {"delta_rule"} | self.rt.product_sources(self.w_in, self.w_gates, self.w_o)
+        return {"delta_rule", "delta_chunk"} | self.rt.product_sources(self.w_in, self.w_gates, self.w_o)
 
     def forward(self, x, ctx, cache):
         H, G, D, Dv, T = self.num_heads, self.num_kv_heads, self.dim, self.vdim, ctx.num_tokens
@@ -135,18 +138,32 @@ class HeadDelta(ChannelDelta):
         proj = self.rt.linear(x, self.w_in)
         gates = self.rt.linear(x, self.w_gates, None, out_dtype=torch.float32)               # [a: H | b: H]
         f32 = lambda n: self.rt.empty(T, n, dtype=torch.float32)
-        qn, kn, vn, beta, decay, kq = f32(G * D), f32(G * D), f32(H * Dv), f32(H), f32(H), f32(G)
+        qn, kn, vn, beta, decay, log_decay, kq = f32(G * D), f32(G * D), f32(H * Dv), f32(H), f32(H), f32(H), f32(G)
         ops.delta_prepare(proj, gates, self.conv, conv_state, ctx.token_row, ctx.row_q_start, ctx.state_slots, self.a_log, self.dt_bias,
-                          qn, kn, vn, beta, decay, kq, num_heads=H, num_kv_heads=G, dim=D, vdim=Dv, unit_eps=self.unit_eps, per_head=True)
+                          qn, kn, vn, beta, decay, kq, num_heads=H, num_kv_heads=G, dim=D, vdim=Dv, unit_eps=self.unit_eps, per_head=True,
+                          log_decay=log_decay)
         if self.taps > 1:
             ops.conv_state_update(proj, ctx.row_q_start, ctx.row_q_len, ctx.state_slots, conv_state)
         o = f32(H * Dv)
-        ops.delta_scan(qn, kn, vn, beta, decay, kq, ctx.row_q_start, ctx.row_q_len, ctx.state_slots, state, o, num_heads=H,
-                       num_kv_heads=G, dim=D, vdim=Dv)
+        self.recurrence(qn, kn, vn, beta, decay, log_decay, kq, ctx, state, o)
         gated = self.rt.empty(T, H * Dv)
         at = 2 * G * D + H * Dv
         ops.head_norm_gate(o, proj[:, at:at + H * Dv], self.norm, gated, H, Dv, self.eps, silu=True)
         return self.rt.linear(gated, self.w_o, None, out_dtype=torch.float32)
+
+
+    def recurrence(self, qn, kn, vn, beta, decay, log_decay, kq, ctx, state, o):
+        """Long portions in chunks, short ones token by token; where the host does not know the rows' lengths (a captured step) each of
+        the two kernels takes the rows that are its own."""
+        sizes = dict(num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, dim=self.dim, vdim=self.vdim)
+        rows = (ctx.row_q_start, ctx.row_q_len, ctx.state_slots, state, o)
+        least = CHUNKED_FROM if ops.delta_chunks_take(self.dim) and ctx.max_q_len >= CHUNKED_FROM else 1 << 30
+        q_lens = ctx.host.get("q_len")
+        long = [n for n in q_lens if n >= least] if q_lens is not None and ctx.max_q_len >= least else None
+        if ctx.max_q_len >= least:
+            ops.delta_chunks(qn, kn, vn, beta, log_decay, *rows, min_len=least, work=(len(long), sum(long)) if long else None, **sizes)
+        if long is None or len(long) < len(q_lens):
+            ops.delta_scan(qn, kn, vn, beta, decay, kq, *rows, below=least, **sizes)
 
 
 register_part("mixer", "head_delta", HeadDelta)
