@@ -38,8 +38,7 @@ __device__ __forceinline__ float conv_at(const T* __restrict__ x, int64_t stride
 }
 
 // proj[t] = [ q: G x D | k: G x D | v: H x Dv | beta logits: H | ... ] (activation type, row stride `stride`);
-// low[t] = [ a: H x A | ... ] float32 (row stride low_stride), A decays a head: D, or 1 -- then the beta logits are float32 too and
-// stand behind them, low[t] = [ a: H | beta logits: H | ... ].  One block per token, one warp per head of q, k or v.
+// low[t] = [ a: H x D | ... ] float32 (row stride low_stride).  One block per token, one warp per head of q, k or v.
 template <typename T>
 __global__ void delta_prepare_kernel(const T* __restrict__ proj, int64_t stride, const float* __restrict__ low, int64_t low_stride,
                                      const float* __restrict__ taps, const float* __restrict__ conv_state,
@@ -47,10 +46,9 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int64_t stride,
                                      const int* __restrict__ state_slots, const float* __restrict__ a_log,
                                      const float* __restrict__ dt_bias, float* __restrict__ qn, float* __restrict__ kn,
                                      float* __restrict__ vn, float* __restrict__ beta, float* __restrict__ decay,
-                                     float* __restrict__ kq, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps, int per_head,
-                                     float* __restrict__ log_decay) {
+                                     float* __restrict__ kq, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps) {
     pdl_enter();
-    const int t = blockIdx.x, A = per_head ? 1 : D;
+    const int t = blockIdx.x;
     const int row = token_row[t];
     const int local = t - row_q_start[row];
     const int C = 2 * G * D + H * Dv;
@@ -91,16 +89,10 @@ __global__ void delta_prepare_kernel(const T* __restrict__ proj, int64_t stride,
         }
     }
     const T* bl = proj + (int64_t)t * stride + C;
-    const float* lo = low + (int64_t)t * low_stride;
-    for (int h = threadIdx.x; h < H; h += blockDim.x) {
-        const float z = per_head ? lo[H + h] : to_f32<T>(bl[h]);
-        beta[(int64_t)t * H + h] = 1.0f / (1.0f + expf(-z));
-    }
-    for (int i = threadIdx.x; i < H * A; i += blockDim.x) {
-        const float rate = expf(a_log[i / A]), ld = -rate * softplus_f(lo[i] + dt_bias[i]);
-        decay[(int64_t)t * H * A + i] = expf(ld);
-        // (e^-100 is nothing in 32 bits; the bound keeps sums of log decays, and their differences, exact to a few parts in a million)
-        if (log_decay) log_decay[(int64_t)t * H * A + i] = fmaxf(ld, -100.f);
+    for (int h = threadIdx.x; h < H; h += blockDim.x) beta[(int64_t)t * H + h] = 1.0f / (1.0f + expf(-to_f32<T>(bl[h])));
+    for (int i = threadIdx.x; i < H * D; i += blockDim.x) {
+        const float rate = expf(a_log[i / D]);
+        decay[(int64_t)t * H * D + i] = expf(-rate * softplus_f(low[(int64_t)t * low_stride + i] + dt_bias[i]));
     }
     __syncthreads();                                   // q and k of this token, written above by other warps of the block
     for (int g = warp; g < G; g += nw) {               // k . q per key head: the same for every value column of the recurrence
@@ -348,8 +340,8 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const TG* __r
 extern "C" int mie_delta_prepare(const void* proj, int tag, long long stride, const float* low, long long low_stride, const float* taps,
                                  const float* conv_state, const int* token_row, const int* row_q_start, const int* state_slots,
                                  const float* a_log, const float* dt_bias, float* qn, float* kn, float* vn, float* beta, float* decay,
-                                 float* kq, int num_tokens, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps, int per_head,
-                                 float* log_decay, cudaStream_t stream) {
+                                 float* kq, int num_tokens, int H, int G, int D, int Dv, int K, float q_scale, float unit_eps,
+                                 cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || Dv <= 0 || K < 1) return MIE_ERR_BAD_ARG;
     const int units = 2 * G + H;
@@ -357,11 +349,11 @@ extern "C" int mie_delta_prepare(const void* proj, int tag, long long stride, co
     if (tag == MIE_F32)
         return launch_kernel(delta_prepare_kernel<float>, dim3(num_tokens), dim3(threads), 0, stream, (const float*)proj, (int64_t)stride,
                              low, (int64_t)low_stride, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias, qn, kn, vn,
-                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps, per_head, log_decay);
+                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps);
     else if (tag == MIE_BF16)
         return launch_kernel(delta_prepare_kernel<bf16>, dim3(num_tokens), dim3(threads), 0, stream, (const bf16*)proj, (int64_t)stride,
                              low, (int64_t)low_stride, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias, qn, kn, vn,
-                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps, per_head, log_decay);
+                             beta, decay, kq, H, G, D, Dv, K, q_scale, unit_eps);
     return MIE_ERR_BAD_ARG;
 }
 

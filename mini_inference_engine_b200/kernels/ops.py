@@ -1183,28 +1183,23 @@ def diff_combine(maps: torch.Tensor, gate, out: torch.Tensor, *, num_heads: int,
 # --------------------------------------------------------------------------- gated delta rule
 
 def delta_prepare(proj: torch.Tensor, low: torch.Tensor, taps, conv_state, token_row, row_q_start, state_slots, a_log, dt_bias,
-                  qn, kn, vn, beta, decay, kq, *, num_heads: int, num_kv_heads: int, dim: int, vdim: int, unit_eps: float,
-                  per_head: bool = False, log_decay=None) -> None:
+                  qn, kn, vn, beta, decay, kq, *, num_heads: int, num_kv_heads: int, dim: int, vdim: int, unit_eps: float) -> None:
     """From rows [q: G x dim | k: G x dim | v: H x vdim | beta logits: H | ...] of the input projection and float32 rows
     [a: H x dim | ...] of the low-rank one: convolution over time + silu of q, k, v (float32 taps [channels, K], older inputs
     from ``conv_state`` [slots, K - 1, channels]), q and k unit vectors per head (q times dim^-1/2), beta = sigmoid,
-    decay = exp(-exp(a_log[h]) softplus(a + dt_bias)), kq = k . q per key head.  All outputs float32.  ``per_head``: one decay per head (``decay`` [T, H]);
-    the float32 rows are [a: H | beta logits: H | ...] and the projection's hold q, k and v only.  ``log_decay``: the decays'
-    logarithms too, none below -100 (float32, of ``decay``'s shape)."""
+    decay = exp(-exp(a_log[h]) softplus(a + dt_bias)), kq = k . q per key head.  All outputs float32."""
     T = proj.shape[0]
     H, G, D, Dv = num_heads, num_kv_heads, dim, vdim
     C = 2 * G * D + H * Dv
     K = taps.shape[1]
-    A = 1 if per_head else D                                         # decays a head
-    _need(proj.dim() == 2 and proj.stride(1) == 1 and proj.shape[1] >= C + (0 if per_head else H), "projection rows must hold q, k, v and beta")
-    _need(low.dtype == torch.float32 and low.stride(1) == 1 and low.shape[0] == T and low.shape[1] >= (2 * H if per_head else H * D),
-          "the decays' rows must be float32")
+    _need(proj.dim() == 2 and proj.stride(1) == 1 and proj.shape[1] >= C + H, "projection rows must hold q, k, v and beta")
+    _need(low.dtype == torch.float32 and low.stride(1) == 1 and low.shape[0] == T and low.shape[1] >= H * D, "low-rank rows must be float32")
     _f32(taps, "taps", C * K)
     _need(conv_state.dtype == torch.float32 and conv_state.is_contiguous() and tuple(conv_state.shape[1:]) == (max(K - 1, 0), C),
           "convolution state must be float32 [slots, K - 1, channels]")
     _f32(a_log, "A_log", H)
-    _f32(dt_bias, "dt_bias", H * A)
-    for t, n in ((qn, G * D), (kn, G * D), (vn, H * Dv), (beta, H), (decay, H * A), (kq, G)):
+    _f32(dt_bias, "dt_bias", H * D)
+    for t, n in ((qn, G * D), (kn, G * D), (vn, H * Dv), (beta, H), (decay, H * D), (kq, G)):
         _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n), "outputs must be float32 [T, n]")
     for t, n in ((token_row, "token_row"), (row_q_start, "row_q_start"), (state_slots, "state_slots")):
         _i32(t, n)
@@ -1212,7 +1207,7 @@ def delta_prepare(proj: torch.Tensor, low: torch.Tensor, taps, conv_state, token
     _check(lib.mie_delta_prepare(_ptr(proj), tag(proj), ctypes.c_longlong(proj.stride(0)), _ptr(low), ctypes.c_longlong(low.stride(0)),
                                  _ptr(taps), _ptr(conv_state), _ptr(token_row), _ptr(row_q_start), _ptr(state_slots), _ptr(a_log),
                                  _ptr(dt_bias), _ptr(qn), _ptr(kn), _ptr(vn), _ptr(beta), _ptr(decay), _ptr(kq), T, H, G, D, Dv, K,
-                                 ctypes.c_float(D ** -0.5), ctypes.c_float(unit_eps), int(per_head), _ptr(log_decay), _stream()), "delta_prepare")
+                                 ctypes.c_float(D ** -0.5), ctypes.c_float(unit_eps), _stream()), "delta_prepare")
 
 
 def conv_state_update(x: torch.Tensor, row_q_start, row_q_len, state_slots, conv_state) -> None:
@@ -1245,6 +1240,73 @@ def delta_scan(qn, kn, vn, beta, decay, kq, row_q_start, row_q_len, state_slots,
     lib = load("delta_rule")
     _check(lib.mie_delta_scan(_ptr(qn), _ptr(kn), _ptr(vn), _ptr(beta), _ptr(decay), _ptr(kq), _ptr(row_q_start), _ptr(row_q_len),
                               _ptr(state_slots), _ptr(state), _ptr(out), row_q_len.numel(), H, G, D, Dv, A, int(below), _stream()), "delta_scan")
+    return out
+
+
+def _head_rows(proj, taps, ring, H, G, D, Dv):
+    C, K = 2 * G * D + H * Dv, taps.shape[0]
+    _need(proj.dtype == torch.float32 and proj.dim() == 2 and proj.stride(1) == 1 and proj.shape[1] >= C + H * Dv + 2 * H,
+          "projection rows must be float32 [q | k | v | gate | a | b]")
+    _f32(taps, "taps", K * C)
+    _need(ring.dtype == torch.float32 and ring.is_contiguous() and tuple(ring.shape[1:]) == (K if K > 1 else 0, C), "convolution ring must be float32 [slots, K, channels]")
+    return C, K
+
+
+def delta_head_prepare(proj: torch.Tensor, taps, ring, positions, token_row, row_q_start, state_slots, a_log, dt_bias, qn, kn, vn, beta, decay,
+                       log_decay, kq, *, num_heads: int, num_kv_heads: int, dim: int, vdim: int, unit_eps: float) -> None:
+    """From float32 rows [q: G x dim | k: G x dim | v: H x vdim | gate: H x vdim | a: H | b: H | ...]: convolution over time + silu of q, k, v
+    (taps [K, channels]; inputs before the step from ``ring`` [slots, K, channels], entry position mod K), q and k unit vectors per
+    head (q times dim^-1/2), beta = sigmoid(b), decay = exp(log_decay), log_decay = -exp(a_log) softplus(a + dt_bias) (none below -100),
+    kq = k . q per key head.  All outputs float32."""
+    T = proj.shape[0]
+    H, G, D, Dv = num_heads, num_kv_heads, dim, vdim
+    _, K = _head_rows(proj, taps, ring, H, G, D, Dv)
+    _f32(a_log, "A_log", H)
+    _f32(dt_bias, "dt_bias", H)
+    for t, n in ((qn, G * D), (kn, G * D), (vn, H * Dv), (beta, H), (decay, H), (log_decay, H), (kq, G)):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n), "outputs must be float32 [T, n]")
+    for t, n in ((positions, "positions"), (token_row, "token_row"), (row_q_start, "row_q_start"), (state_slots, "state_slots")):
+        _i32(t, n)
+    _check(load("delta_head").mie_delta_head_prepare(_ptr(proj), ctypes.c_longlong(proj.stride(0)), _ptr(taps), _ptr(ring), _ptr(positions), _ptr(token_row),
+                                                     _ptr(row_q_start), _ptr(state_slots), _ptr(a_log), _ptr(dt_bias), _ptr(qn), _ptr(kn), _ptr(vn),
+                                                     _ptr(beta), _ptr(decay), _ptr(log_decay), _ptr(kq), T, H, G, D, Dv, K, ctypes.c_float(D ** -0.5),
+                                                     ctypes.c_float(unit_eps), _stream()), "delta_head_prepare")
+
+
+def delta_head_remember(proj: torch.Tensor, ring, positions, row_q_start, row_q_len, state_slots, *, num_heads: int, num_kv_heads: int, dim: int,
+                        vdim: int) -> None:
+    """The last K - 1 inputs of every row's portion into its ``ring``."""
+    K = ring.shape[1]
+    _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and ring.dtype == torch.float32 and ring.is_contiguous()
+          and ring.shape[2] == 2 * num_kv_heads * dim + num_heads * vdim <= proj.shape[1], "float32 rows and ring of the channels")
+    for t, n in ((positions, "positions"), (row_q_start, "row_q_start"), (row_q_len, "row_q_len"), (state_slots, "state_slots")):
+        _i32(t, n)
+    _check(load("delta_head").mie_delta_head_remember(_ptr(proj), ctypes.c_longlong(proj.stride(0)), _ptr(ring), _ptr(positions), _ptr(row_q_start),
+                                                      _ptr(row_q_len), _ptr(state_slots), row_q_len.numel(), num_heads, num_kv_heads, dim, vdim, K,
+                                                      _stream()), "delta_head_remember")
+
+
+def delta_head_step_takes(dim: int, vdim: int) -> bool:
+    """Whether ``delta_head_step`` serves heads of this size (a head's state must fit in shared memory)."""
+    return dim * vdim <= 51200 and load("delta_head").mie_delta_head_step_bytes(dim, vdim) <= 200 * 1024
+
+
+def delta_head_step(proj: torch.Tensor, taps, ring, positions, row_q_start, row_q_len, state_slots, a_log, dt_bias, state, norm, out: torch.Tensor, *,
+                    num_heads: int, num_kv_heads: int, dim: int, vdim: int, unit_eps: float, eps: float) -> torch.Tensor:
+    """The whole delta rule of rows with one new token -- ``delta_head_prepare``, the recurrence, the ring, the heads' norm with weight ``norm``
+    [vdim] and the gate silu(gate) -- in one launch.  ``out`` [T, H * vdim]; other rows are left alone."""
+    H, G, D, Dv = num_heads, num_kv_heads, dim, vdim
+    _, K = _head_rows(proj, taps, ring, H, G, D, Dv)
+    for t, n, name in ((a_log, H, "A_log"), (dt_bias, H, "dt_bias"), (norm, Dv, "head norm weight")):
+        _f32(t, name, n)
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, Dv, D), "state must be float32 [slots, H, vdim, dim]")
+    _need(out.is_contiguous() and out.shape == (proj.shape[0], H * Dv), "out must be contiguous [T, H * vdim]")
+    for t, n in ((positions, "positions"), (row_q_start, "row_q_start"), (row_q_len, "row_q_len"), (state_slots, "state_slots")):
+        _i32(t, n)
+    _check(load("delta_head").mie_delta_head_step(_ptr(proj), ctypes.c_longlong(proj.stride(0)), _ptr(taps), _ptr(ring), _ptr(positions), _ptr(row_q_start),
+                                                  _ptr(row_q_len), _ptr(state_slots), _ptr(a_log), _ptr(dt_bias), _ptr(state), _ptr(norm), _ptr(out),
+                                                  tag(out), row_q_len.numel(), H, G, D, Dv, K, ctypes.c_float(D ** -0.5), ctypes.c_float(unit_eps),
+                                                  ctypes.c_float(eps), _stream()), "delta_head_step")
     return out
 
 

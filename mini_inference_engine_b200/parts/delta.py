@@ -67,10 +67,7 @@ class ChannelDelta(Mixer):
         up[H * D:, ra:ra + rg] = g2
         self.w_up = rt.place(up)
         self.w_o = rt.place(tensors["o"])
-        self.bind_small(tensors)
-
-    def bind_small(self, tensors):
-        small = lambda t: t.float().to(self.rt.device).contiguous()          # read as float32 by the kernels
+        small = lambda t: t.float().to(rt.device).contiguous()               # read as float32 by the kernels
         self.conv = small(torch.cat([tensors["q.conv"].float(), tensors["k.conv"].float(), tensors["v.conv"].float()], 0))
         self.a_log, self.dt_bias, self.norm = small(tensors["A_log"]), small(tensors["dt_bias"]), small(tensors["norm"])
 
@@ -106,64 +103,79 @@ register_part("mixer", "channel_delta", ChannelDelta)
 CHUNKED_FROM = 40        # new tokens from which a row's recurrence goes in chunks
 
 
-class HeadDelta(ChannelDelta):
+class HeadDelta(Mixer):
     """The gated delta rule with ONE decay per head, g = exp(-exp(A_log_h) softplus(W_a h + dt_bias)_h), and an output gate silu(W_g h) laid
-    out heads x vdim; everything else as ``ChannelDelta``.  q|k|v|g of the input are one product; a|b, which decide decays and
-    step sizes, a second one that leaves float32."""
+    out heads x vdim; everything else as ``ChannelDelta``.
+
+    q|k|v|g|a|b of the input are one product that leaves float32 (a and b decide decays and step sizes).  A step of single tokens is one
+    kernel between the two products.  Portions: convolution, activations, unit vectors and decays are one kernel, the recurrence
+    goes in chunks where a row is long enough and token by token where it is not, head norm and gate are one more.  Two states: S
+    [heads, vdim, dim] and the convolution's inputs as a ring over positions [taps, channels]."""
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, taps: int, eps: float, unit_eps: float = 1e-6):
-        super().__init__(hidden_size, num_heads, num_kv_heads, dim, vdim, taps, eps, unit_eps=unit_eps)
+        if num_heads % num_kv_heads:
+            raise ValueError("num_heads must be a multiple of num_kv_heads")
+        if taps < 1:
+            raise ValueError("the convolution has at least one tap")
+        if dim > 512:
+            raise ValueError(f"key size {dim}: the recurrence kernels take up to 512")
+        self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim = hidden_size, num_heads, num_kv_heads, dim, vdim
+        self.taps, self.eps, self.unit_eps = taps, eps, unit_eps
 
     def tensor_specs(self):
-        H, Dv, h = self.num_heads, self.vdim, self.hidden_size
-        specs = {n: s for n, s in super().tensor_specs().items() if n not in ("a1", "a2", "g1", "g2")}
-        specs.update({"a": TensorSpec((H, h), "fan_in"), "dt_bias": TensorSpec((H,), "uniform:-4:1"), "g": TensorSpec((H * Dv, h), "fan_in")})
-        return specs
+        H, G, D, Dv, h, K = self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.hidden_size, self.taps
+        return {"q": TensorSpec((G * D, h), "fan_in"), "q.conv": TensorSpec((G * D, K), "normal:0:0.5"),
+                "k": TensorSpec((G * D, h), "fan_in"), "k.conv": TensorSpec((G * D, K), "normal:0:0.5"),
+                "v": TensorSpec((H * Dv, h), "fan_in"), "v.conv": TensorSpec((H * Dv, K), "normal:0:0.5"),
+                "b": TensorSpec((H, h), "fan_in"), "a": TensorSpec((H, h), "fan_in"), "A_log": TensorSpec((H,), "uniform:-3:0.5"),
+                "dt_bias": TensorSpec((H,), "uniform:-4:1"), "norm": TensorSpec((Dv,), "normal:1:0.1"), "g": TensorSpec((H * Dv, h), "fan_in"),
+                "o": TensorSpec((h, H * Dv), "fan_in")}
 
     def bind(self, tensors, rt):
         self.rt = rt
-        w, _ = _padded_rows([tensors[n] for n in ("q", "k", "v", "g")])
+        w, _ = _padded_rows([tensors[n] for n in ("q", "k", "v", "g", "a", "b")])
         self.w_in = rt.place(w)
-        w, _ = _padded_rows([tensors["a"], tensors["b"]])
-        self.w_gates = rt.place(w)
         self.w_o = rt.place(tensors["o"])
-        self.bind_small(tensors)
+        small = lambda t: t.float().to(rt.device).contiguous()               # read as float32 by the kernels
+        self.conv = small(torch.cat([tensors[n + ".conv"].float() for n in "qkv"], 0).t())          # [taps, channels]
+        self.a_log, self.dt_bias, self.norm = small(tensors["A_log"]), small(tensors["dt_bias"]), small(tensors["norm"])
+
+    def cache_need(self):
+        C = 2 * self.num_kv_heads * self.dim + self.num_heads * self.vdim
+        return (StateNeed((self.num_heads, self.vdim, self.dim), torch.float32), StateNeed((self.taps if self.taps > 1 else 0, C), torch.float32))
 
     def kernel_sources(self):
-        return {"delta_rule", "delta_chunk"} | self.rt.product_sources(self.w_in, self.w_gates, self.w_o)
+        return {"delta_rule", "delta_chunk", "delta_head"} | self.rt.product_sources(self.w_in, self.w_o)
 
     def forward(self, x, ctx, cache):
+        from ..kernels.attention import decode_only
         H, G, D, Dv, T = self.num_heads, self.num_kv_heads, self.dim, self.vdim, ctx.num_tokens
-        state, conv_state = cache.parts[0].state, cache.parts[1].state
-        proj = self.rt.linear(x, self.w_in)
-        gates = self.rt.linear(x, self.w_gates, None, out_dtype=torch.float32)               # [a: H | b: H]
-        f32 = lambda n: self.rt.empty(T, n, dtype=torch.float32)
-        qn, kn, vn, beta, decay, log_decay, kq = f32(G * D), f32(G * D), f32(H * Dv), f32(H), f32(H), f32(H), f32(G)
-        ops.delta_prepare(proj, gates, self.conv, conv_state, ctx.token_row, ctx.row_q_start, ctx.state_slots, self.a_log, self.dt_bias,
-                          qn, kn, vn, beta, decay, kq, num_heads=H, num_kv_heads=G, dim=D, vdim=Dv, unit_eps=self.unit_eps, per_head=True,
-                          log_decay=log_decay)
-        if self.taps > 1:
-            ops.conv_state_update(proj, ctx.row_q_start, ctx.row_q_len, ctx.state_slots, conv_state)
-        o = f32(H * Dv)
-        self.recurrence(qn, kn, vn, beta, decay, log_decay, kq, ctx, state, o)
+        state, ring = cache.parts[0].state, cache.parts[1].state
+        sizes = dict(num_heads=H, num_kv_heads=G, dim=D, vdim=Dv)
+        proj = self.rt.linear(x, self.w_in, None, out_dtype=torch.float32)
         gated = self.rt.empty(T, H * Dv)
+        if decode_only(ctx) and ops.delta_head_step_takes(D, Dv):
+            ops.delta_head_step(proj, self.conv, ring, ctx.positions, ctx.row_q_start, ctx.row_q_len, ctx.state_slots, self.a_log, self.dt_bias, state,
+                                self.norm, gated, unit_eps=self.unit_eps, eps=self.eps, **sizes)
+            return self.rt.linear(gated, self.w_o, None, out_dtype=torch.float32)
+        f32 = lambda n: self.rt.empty(T, n, dtype=torch.float32)
+        qn, kn, vn, beta, decay, log_decay, kq, o = f32(G * D), f32(G * D), f32(H * Dv), f32(H), f32(H), f32(H), f32(G), f32(H * Dv)
+        ops.delta_head_prepare(proj, self.conv, ring, ctx.positions, ctx.token_row, ctx.row_q_start, ctx.state_slots, self.a_log, self.dt_bias,
+                               qn, kn, vn, beta, decay, log_decay, kq, unit_eps=self.unit_eps, **sizes)
+        if self.taps > 1:
+            ops.delta_head_remember(proj, ring, ctx.positions, ctx.row_q_start, ctx.row_q_len, ctx.state_slots, **sizes)
+        rows = (ctx.row_q_start, ctx.row_q_len, ctx.state_slots, state, o)
+        # where the host does not know the rows' lengths (a captured step) each of the two kernels takes the rows that are its own
+        chunked = ops.delta_chunks_take(D) and ctx.max_q_len >= CHUNKED_FROM
+        q_lens = ctx.host.get("q_len")
+        long = [n for n in q_lens if n >= CHUNKED_FROM] if chunked and q_lens is not None else None
+        if chunked:
+            ops.delta_chunks(qn, kn, vn, beta, log_decay, *rows, min_len=CHUNKED_FROM, work=(len(long), sum(long)) if long else None, **sizes)
+        if long is None or len(long) < len(q_lens):
+            ops.delta_scan(qn, kn, vn, beta, decay, kq, *rows, below=CHUNKED_FROM if chunked else 1 << 30, **sizes)
         at = 2 * G * D + H * Dv
         ops.head_norm_gate(o, proj[:, at:at + H * Dv], self.norm, gated, H, Dv, self.eps, silu=True)
         return self.rt.linear(gated, self.w_o, None, out_dtype=torch.float32)
-
-
-    def recurrence(self, qn, kn, vn, beta, decay, log_decay, kq, ctx, state, o):
-        """Long portions in chunks, short ones token by token; where the host does not know the rows' lengths (a captured step) each of
-        the two kernels takes the rows that are its own."""
-        sizes = dict(num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, dim=self.dim, vdim=self.vdim)
-        rows = (ctx.row_q_start, ctx.row_q_len, ctx.state_slots, state, o)
-        least = CHUNKED_FROM if ops.delta_chunks_take(self.dim) and ctx.max_q_len >= CHUNKED_FROM else 1 << 30
-        q_lens = ctx.host.get("q_len")
-        long = [n for n in q_lens if n >= least] if q_lens is not None and ctx.max_q_len >= least else None
-        if ctx.max_q_len >= least:
-            ops.delta_chunks(qn, kn, vn, beta, log_decay, *rows, min_len=least, work=(len(long), sum(long)) if long else None, **sizes)
-        if long is None or len(long) < len(q_lens):
-            ops.delta_scan(qn, kn, vn, beta, decay, kq, *rows, below=least, **sizes)
 
 
 register_part("mixer", "head_delta", HeadDelta)
