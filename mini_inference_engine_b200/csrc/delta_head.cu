@@ -37,26 +37,41 @@ template <int VEC> __device__ __forceinline__ void store_vec(float* p, const flo
 }
 
 // VEC channels from c on of token t, `local` tokens into its row's portion, at position `pos`: the convolution's output behind silu.
-template <int VEC>
+// KT: the number of taps where it is known at compile time (all inputs are then asked for together), 0: p.K.
+template <int VEC, int KT>
 __device__ __forceinline__ void conv_silu(float* y, const HeadParams& p, const float* ring_slot, int t, int local, int pos, int c) {
-    const int C = 2 * p.G * p.D + p.H * p.Dv, m = p.K > 1 ? pos % p.K : 0;
+    const int K = KT > 0 ? KT : p.K, C = 2 * p.G * p.D + p.H * p.Dv, m = K > 1 ? pos % K : 0;
 #pragma unroll
     for (int e = 0; e < VEC; ++e) y[e] = 0.f;
-    for (int back = p.K - 1; back >= 0; --back) {
-        float x[VEC], w[VEC];
-        load_vec<VEC>(w, p.taps + (int64_t)(p.K - 1 - back) * C + c);
+    auto input = [&](float* x, int back) {
         int entry = m - back;
-        if (entry < 0) entry += p.K;
+        if (entry < 0) entry += K;
         load_vec<VEC>(x, back <= local ? p.proj + (int64_t)(t - back) * p.stride + c : ring_slot + (int64_t)entry * C + c);
+    };
+    auto add = [&](const float* x, const float* w) {
 #pragma unroll
         for (int e = 0; e < VEC; ++e) y[e] = fmaf(w[e], x[e], y[e]);
+    };
+    if constexpr (KT > 0) {
+        float x[KT][VEC], w[KT][VEC];
+#pragma unroll
+        for (int i = 0; i < KT; ++i) { input(x[i], KT - 1 - i); load_vec<VEC>(w[i], p.taps + (int64_t)i * C + c); }
+#pragma unroll
+        for (int i = 0; i < KT; ++i) add(x[i], w[i]);
+    } else {
+        for (int i = 0; i < K; ++i) {
+            float x[VEC], w[VEC];
+            input(x, K - 1 - i);
+            load_vec<VEC>(w, p.taps + (int64_t)i * C + c);
+            add(x, w);
+        }
     }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) y[e] = silu_of(y[e]);
 }
 
 // Work items of a token: G heads of q and k together, H heads of v, and one for the gates.  NCH: pieces of 32 * VEC channels a key head.
-template <int VEC, int NCH>
+template <int VEC, int NCH, int KT>
 __global__ void __launch_bounds__(256) delta_head_prepare_kernel(const HeadParams p, float* __restrict__ qn, float* __restrict__ kn, float* __restrict__ vn,
                                                                  float* __restrict__ beta, float* __restrict__ decay, float* __restrict__ log_decay,
                                                                  float* __restrict__ kq, int num_tokens, int tile) {
@@ -83,7 +98,7 @@ __global__ void __launch_bounds__(256) delta_head_prepare_kernel(const HeadParam
             const int h = unit - G;
             for (int d = lane * VEC; d < Dv; d += 32 * VEC) {
                 float y[VEC];
-                conv_silu<VEC>(y, p, ring_slot, t, local, pos, 2 * G * D + h * Dv + d);
+                conv_silu<VEC, KT>(y, p, ring_slot, t, local, pos, 2 * G * D + h * Dv + d);
                 store_vec<VEC>(vn + ((int64_t)t * H + h) * Dv + d, y);
             }
             continue;
@@ -95,8 +110,8 @@ __global__ void __launch_bounds__(256) delta_head_prepare_kernel(const HeadParam
 #pragma unroll
             for (int e = 0; e < VEC; ++e) q[n][e] = k[n][e] = 0.f;
             if (d < D) {
-                conv_silu<VEC>(q[n], p, ring_slot, t, local, pos, unit * D + d);
-                conv_silu<VEC>(k[n], p, ring_slot, t, local, pos, (G + unit) * D + d);
+                conv_silu<VEC, KT>(q[n], p, ring_slot, t, local, pos, unit * D + d);
+                conv_silu<VEC, KT>(k[n], p, ring_slot, t, local, pos, (G + unit) * D + d);
             }
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
@@ -141,7 +156,7 @@ __device__ __forceinline__ void copy_async(float* dst, const float* src, int byt
 #define STEP_THREADS 256
 
 // One new token a row.  VEC entries of a column of the state go together; eight lanes share a column, NM pieces each.
-template <typename T, int VEC, int NM>
+template <typename T, int VEC, int NM, int KT>
 __global__ void __launch_bounds__(STEP_THREADS) delta_head_step_kernel(const HeadParams p, float* __restrict__ state, const float* __restrict__ norm,
                                                                        T* __restrict__ out, float eps) {
     extern __shared__ __align__(16) float sm[];
@@ -169,7 +184,7 @@ __global__ void __launch_bounds__(STEP_THREADS) delta_head_step_kernel(const Hea
         const int seg = i < D ? 0 : i < 2 * D ? 1 : 2;
         const int d = i - seg * D, c = seg == 0 ? g * D + d : seg == 1 ? (G + g) * D + d : 2 * G * D + h * Dv + d;
         float y[VEC], in[VEC];
-        conv_silu<VEC>(y, p, ring_slot, t, 0, pos, c);
+        conv_silu<VEC, KT>(y, p, ring_slot, t, 0, pos, c);
         store_vec<VEC>((seg == 0 ? q : seg == 1 ? k : v) + d, y);
         if (p.K > 1 && (seg == 2 || keeps_keys)) {
             load_vec<VEC>(in, x + c);
@@ -265,10 +280,11 @@ extern "C" int mie_delta_head_prepare(const float* proj, long long stride, const
     if (rc) return rc;
     const int tile = num_tokens >= 512 ? 8 : num_tokens >= 128 ? 2 : 1;
     const dim3 grid((num_tokens + tile - 1) / tile, (G + H + 1 + 7) / 8);
-#define PREPARE(VEC, NCH) launch_kernel(delta_head_prepare_kernel<VEC, NCH>, grid, dim3(256), 0, stream, p, qn, kn, vn, beta, decay, log_decay, kq, num_tokens, tile)
+#define PREPARE(VEC, NCH, KT) launch_kernel(delta_head_prepare_kernel<VEC, NCH, KT>, grid, dim3(256), 0, stream, p, qn, kn, vn, beta, decay, log_decay, kq, num_tokens, tile)
     const bool vec = head_vec(p) && ((reinterpret_cast<uintptr_t>(qn) | reinterpret_cast<uintptr_t>(kn) | reinterpret_cast<uintptr_t>(vn)) & 15) == 0;
-    if (vec) return D <= 128 ? PREPARE(4, 1) : D <= 256 ? PREPARE(4, 2) : PREPARE(4, 4);
-    return D <= 128 ? PREPARE(1, 4) : PREPARE(1, 16);
+    if (vec && D <= 128) return K == 4 ? PREPARE(4, 1, 4) : PREPARE(4, 1, 0);
+    if (vec) return PREPARE(4, 4, 0);
+    return D <= 128 ? PREPARE(1, 4, 0) : PREPARE(1, 16, 0);
 #undef PREPARE
 }
 
@@ -300,17 +316,19 @@ extern "C" int mie_delta_head_step(const float* proj, long long stride, const fl
     const int smem = mie_delta_head_step_bytes(D, Dv);
     if ((int64_t)D * Dv > 51200 || smem > 200 * 1024 || num_rows > 65535) return MIE_ERR_TOO_LARGE;
     const bool vec = head_vec(p) && (reinterpret_cast<uintptr_t>(state) & 15) == 0;
-#define STEP(T, VEC, NM)                                                                                                                          \
+#define STEP(T, VEC, NM, KT)                                                                                                                          \
     do {                                                                                                                                          \
-        const cudaError_t e = cudaFuncSetAttribute(delta_head_step_kernel<T, VEC, NM>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);         \
+        const cudaError_t e = cudaFuncSetAttribute(delta_head_step_kernel<T, VEC, NM, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);         \
         if (e != cudaSuccess) return (int)e;                                                                                                      \
-        return launch_kernel(delta_head_step_kernel<T, VEC, NM>, dim3(H, num_rows), dim3(STEP_THREADS), (size_t)smem, stream, p, state, norm, (T*)out, eps); \
+        return launch_kernel(delta_head_step_kernel<T, VEC, NM, KT>, dim3(H, num_rows), dim3(STEP_THREADS), (size_t)smem, stream, p, state, norm, (T*)out, eps); \
     } while (0)
 #define STEPS(T)                                                                          \
     do {                                                                                  \
-        if (vec) { if (D <= 64) STEP(T, 4, 2); if (D <= 128) STEP(T, 4, 4); STEP(T, 4, 16); } \
-        if (D <= 128) STEP(T, 1, 16);                                                     \
-        STEP(T, 1, 64);                                                                   \
+        if (vec && D <= 128 && K == 4) STEP(T, 4, 4, 4);                                  \
+        if (vec && D <= 128) STEP(T, 4, 4, 0);                                            \
+        if (vec) STEP(T, 4, 16, 0);                                                       \
+        if (D <= 128) STEP(T, 1, 16, 0);                                                  \
+        STEP(T, 1, 64, 0);                                                                   \
     } while (0)
     if (tag == MIE_F32) STEPS(float);
     if (tag == MIE_BF16) STEPS(bf16);
