@@ -74,7 +74,7 @@ struct ChunkScratch {           // per (chunk, head): T diag(beta) [64, 64], P [
 __device__ __forceinline__ int chunks_of(int n, int min_len) { return n >= min_len ? (n + CH - 1) / CH : 0; }
 
 template <int DT>
-__global__ void __launch_bounds__(256) delta_chunk_prep_kernel(const float* __restrict__ qn, const float* __restrict__ kn,
+__global__ void __launch_bounds__(256, 2) delta_chunk_prep_kernel(const float* __restrict__ qn, const float* __restrict__ kn,
                                                                const float* __restrict__ beta, const float* __restrict__ log_decay,
                                                                const int* __restrict__ row_q_start, const int* __restrict__ row_q_len,
                                                                int num_rows, int min_len, float* __restrict__ scratch, int H, int G, int D) {
@@ -83,9 +83,9 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(const float* __re
     float* Q = K + CH * (DT + 4);
     float* KK = Q + CH * (DT + 4);                             // [64][68]: k_i . k_j
     float* QK = KK + CH * CHP;                                 // q_i . k_j
-    float* A = QK + CH * CHP;
-    float* X = K;                                              // products on the way to T, and T: keys and queries are not read after the Gram matrices
-    float* T = Q;                                              // [64][68]
+    float* X = QK + CH * CHP;                                  // products on the way to T [3][16][16]
+    float* A = K;                                              // [64][68], and T: keys and queries are not read after the Gram matrices
+    float* T = Q;
     __shared__ float lg[CH], be[CH];
     __shared__ int s_row, s_chunk;
     pdl_enter();
@@ -182,7 +182,12 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(const float* __re
             for (int idx = threadIdx.x; idx < n; idx += blockDim.x) {
                 const int bi = w + (idx >> 8), bj = bi - w, r = (idx >> 4) & 15, c = idx & 15;
                 float v = 0.f;
-                for (int m = bj * 16; m < bi * 16; ++m) v = fmaf(A[(bi * 16 + r) * CHP + m], T[m * CHP + bj * 16 + c], v);
+                for (int mb = bj * 16; mb < bi * 16; mb += 16) {
+                    float part = 0.f;
+#pragma unroll
+                    for (int m = 0; m < 16; ++m) part = fmaf(A[(bi * 16 + r) * CHP + mb + m], T[(mb + m) * CHP + bj * 16 + c], part);
+                    v += part;
+                }
                 X[idx] = v;
             }
             __syncthreads();
@@ -420,7 +425,7 @@ template <int DT>
 static int launch_chunks(const float* qn, const float* kn, const float* vn, const float* beta, const float* log_decay, const int* row_q_start,
                          const int* row_q_len, const int* state_slots, float* state, float* out, float* scratch, int max_chunks, int num_rows,
                          int min_len, int H, int G, int D, int Dv, cudaStream_t stream) {
-    const size_t prep = (size_t)(2 * CH * (DT + 4) + 3 * CH * CHP) * sizeof(float);
+    const size_t prep = (size_t)(2 * CH * (DT + 4) + 2 * CH * CHP + 3 * 256) * sizeof(float);      // two blocks on an SM
     const size_t scan = (size_t)(2 * (2 * CH * (DT + 4) + CH * COLS + 2 * CH) + 2 * CH * CHP + COLS * (DT + 4) + 3 * COLS * CHP) * sizeof(float);
     cudaError_t e = cudaFuncSetAttribute(delta_chunk_prep_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_scan_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)scan);

@@ -17,7 +17,7 @@
 #include "common.cuh"
 
 __device__ __forceinline__ float softplus_of(float x) { return x > 20.f ? x : log1pf(expf(x)); }
-__device__ __forceinline__ float silu_of(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu_of(float x) { return __fdividef(x, 1.0f + __expf(-fmaxf(x, -80.f))); }      // (the bound keeps the divisor in the fast division's range)
 
 struct HeadParams {
     const float* proj; int64_t stride;

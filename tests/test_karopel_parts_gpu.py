@@ -395,8 +395,11 @@ DELTA = [delta(), delta(1, 1, 48, 8, 1), delta(2, 2, 128, 40, 2), delta(3, 1, 20
 
 
 @pytest.mark.parametrize("dt", DTYPES)
+@pytest.mark.parametrize("chunked_from", [2, 112])
 @pytest.mark.parametrize("case", DELTA)
-def test_delta_rule(dt, case):
+def test_delta_rule(dt, case, chunked_from, monkeypatch):
+    from mini_inference_engine_b200.parts import delta as delta_parts
+    monkeypatch.setattr(delta_parts, "CHUNKED_FROM", chunked_from)
     rt = rt_for(dt)
     params, cfg = case
     mixer = build("mixer", "head_delta", **params)
@@ -408,9 +411,13 @@ def test_delta_rule(dt, case):
 @pytest.mark.parametrize("dt", DTYPES)
 @pytest.mark.parametrize("rate", [-9.0, -2.0, 0.5, 4.0])
 @pytest.mark.parametrize("heads,dim,vdim", [(2, 64, 32), (2, 128, 128), (1, 40, 24)])
-def test_delta_rule_over_long_portions_at_every_rate_of_decay(dt, rate, heads, dim, vdim):
+@pytest.mark.parametrize("chunked_from", [1, 40, 112])
+def test_delta_rule_over_long_portions_at_every_rate_of_decay(dt, rate, heads, dim, vdim, chunked_from, monkeypatch):
     """Portions of several hundred tokens, of lengths around the multiples of 16, 32 and 64, from decays of almost 1 to states that
-    vanish within a token; keys that repeat, so that the corrections of a token by the ones before it are large."""
+    vanish within a token; keys that repeat, so that the corrections of a token by the ones before it are large.  Which portions go
+    in chunks and which token by token makes no difference."""
+    from mini_inference_engine_b200.parts import delta as delta_parts
+    monkeypatch.setattr(delta_parts, "CHUNKED_FROM", chunked_from)
     rt = rt_for(dt)
     params, cfg = delta(heads, 1, dim, vdim, 4)
     mixer = build("mixer", "head_delta", **params)
@@ -466,6 +473,48 @@ def test_a_slot_that_is_used_again_starts_from_zero_and_rows_do_not_mix(dt):
         at += n
     close(torch.cat(ga, 0), plain(a[:25]), dt, "the row that decodes")
     close(torch.cat(gb, 0), plain(b), dt, "the row that takes portions")
+
+
+@pytest.mark.parametrize("groups,dim,vdim,least", [(1, 128, 48, 1), (2, 64, 16, 30), (3, 36, 100, 64)])
+def test_chunks_and_single_steps_of_several_rows_in_one_launch(groups, dim, vdim, least):
+    """The chunked kernel and the token-by-token one share a batch: rows of ``least`` tokens or more and the others, each from a state of its own
+    that is not zero, in slots out of order; both against the plain recurrence, outputs and states."""
+    from mini_inference_engine_b200.kernels import ops
+    H, G, lens, slots = 2 * groups, groups, (70, 1, 128, 29, 30, 64, 200, 3), (5, 2, 8, 1, 7, 3, 4, 6)
+    T = sum(lens)
+    g = torch.Generator().manual_seed(dim)
+    unit = lambda z: z / z.norm(dim=-1, keepdim=True)
+    q, k = unit(torch.randn(T, G, dim, generator=g)) * dim ** -0.5, unit(torch.randn(T, G, dim, generator=g) + 0.7)
+    v, beta = torch.randn(T, H, vdim, generator=g), torch.rand(T, H, generator=g)
+    log_decay = -torch.rand(T, H, generator=g) ** 4
+    state = torch.randn(9, H, vdim, dim, generator=g)
+    want, after, at = torch.zeros(T, H, vdim), state.clone(), 0
+    for n, slot in zip(lens, slots):
+        S = state[slot].double().transpose(1, 2)                       # [H, dim, vdim]
+        for t in range(at, at + n):
+            kk, qq = (z[t].double().repeat_interleave(H // G, 0) for z in (k, q))
+            S = log_decay[t].double().exp()[:, None, None] * S
+            u = beta[t].double()[:, None] * (v[t].double() - torch.einsum("hdv,hd->hv", S, kk))
+            S = S + kk[:, :, None] * u[:, None, :]
+            want[t] = torch.einsum("hdv,hd->hv", S, qq).float()
+        after[slot] = S.transpose(1, 2).float()
+        at += n
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=DEV)
+    d = lambda t: t.reshape(t.shape[0], -1).contiguous().to(DEV)
+    st, out = state.to(DEV), torch.full((T, H * vdim), 7.0, device=DEV)
+    starts = [sum(lens[:i]) for i in range(len(lens))]
+    args = (i32(starts), i32(lens), i32(slots), st, out)
+    sizes = dict(num_heads=H, num_kv_heads=G, dim=dim, vdim=vdim)
+    long = [n for n in lens if n >= least]
+    ops.delta_chunks(d(q), d(k), d(v), d(beta), d(log_decay), *args, min_len=least, work=(len(long), sum(long)) if groups != 2 else None, **sizes)
+    torch.cuda.synchronize()
+    for n, s0, slot in zip(lens, starts, slots):
+        if n < least:
+            assert (out[s0:s0 + n] == 7.0).all() and torch.equal(st[slot].cpu(), state[slot]), "a row below the bound is left alone"
+    kq = (k * q).sum(-1)
+    ops.delta_scan(d(q), d(k), d(v), d(beta), d(log_decay.exp()), d(kq), *args, below=least, **sizes)
+    close_at(out.reshape(T, H, vdim), want, torch.float32, "outputs")
+    close_at(st, after, torch.float32, "states")
 
 
 # ----------------------------------------------------------------------------------------------- side by side
